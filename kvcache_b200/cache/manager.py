@@ -5,7 +5,7 @@ src/include/kv_cache_manager.h:27-92) and the app's own handling
 (apps/qwen_serve.cu:85-93, :134-135), and adds groups: cache entries whose keys
 and values have the same geometry and reach share one block table and one page id,
 as the reference's 24 layers share one (apps/qwen_serve.cu:99-100); entries with
-a window form a group of their own and give pages back once the window has passed.
+a window (or chunks) form a group of their own and give pages back once the window has passed (the chunk is over).
 """
 from __future__ import annotations
 
@@ -56,7 +56,7 @@ class CacheManager:
                 if entry.kv not in by_spec:
                     by_spec[entry.kv] = len(self.groups)
                     self.groups.append(CacheGroup(entry.kv, [], GroupPages(
-                        num_pages, page_size, max_slots, self.max_pages_per_request, entry.kv.window, entry.kv.keep_first)))
+                        num_pages, page_size, max_slots, self.max_pages_per_request, entry.kv.window, entry.kv.keep_first, entry.kv.chunk)))
                 g = by_spec[entry.kv]
                 self.entry_group[cache_id] = (g, len(self.groups[g].cache_ids))
                 self.groups[g].cache_ids.append(cache_id)

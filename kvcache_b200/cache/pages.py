@@ -85,9 +85,10 @@ class GroupPages:
     same geometry and the same reach (all keys, or a window of them) share page ids."""
 
     def __init__(self, num_pages: int, page_size: int, max_slots: int, max_pages_per_request: int,
-                 window: Optional[int] = None, keep_first: int = 0):
+                 window: Optional[int] = None, keep_first: int = 0, chunk: Optional[int] = None):
         self.page_size = page_size
         self.window = window
+        self.chunk = chunk                         # queries see the keys of their own chunk of this many tokens only
         # With a window: the pages of the request's first `keep_first` tokens are never given back before the request ends.
         self.kept_pages = pages_for(keep_first, page_size) if window is not None else 0
         self.allocator = PageAllocator(num_pages)
@@ -101,6 +102,8 @@ class GroupPages:
     # ---- what a range of new positions needs --------------------------------
     def first_needed_page(self, start: int) -> int:
         """First logical page that queries at positions >= start still read."""
+        if self.chunk is not None:
+            return start // self.chunk * self.chunk // self.page_size
         if self.window is None:
             return 0
         return max(0, start - self.window + 1) // self.page_size
@@ -160,7 +163,8 @@ class GroupPages:
         """Most pages a request of `total_tokens` holds at once when no step brings more
         than `largest_portion` of its tokens."""
         full = pages_for(total_tokens, self.page_size)
-        if self.window is None:
+        reach = self.window if self.chunk is None else self.chunk       # a chunk's keys lie within a window of its size
+        if reach is None:
             return full
-        span = self.window - 1 + max(1, largest_portion)
+        span = reach - 1 + max(1, largest_portion)
         return min(full, pages_for(span, self.page_size) + 1 + self.kept_pages)

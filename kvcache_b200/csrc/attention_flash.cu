@@ -67,7 +67,7 @@ __global__ void __launch_bounds__(128) flash_decode_kernel(const DecodeParams p)
     const int q_start = p.seg_q_start[seg], q_len = p.seg_q_len[seg], kv_len = p.seg_kv_len[seg];
     const int rows = min(q_len * G, 16);   // an item is one warp tile of 16 rows; rows beyond it are not this kernel's (see no_alloc.h)
     const int first_pos = kv_len - q_len;
-    const int key_lo = (p.window > 0 && first_pos - p.window + 1 > 0) ? first_pos - p.window + 1 : 0;
+    const int key_lo = first_seen_key(first_pos, p.window), lo_max = first_seen_key(kv_len - 1, p.window);
     const int tile_end = (kv_len + KT - 1) / KT;
     const int keep = p.window > 0 ? p.keep : 0;
     const TileList tl(key_lo, tile_end, keep);                         // positions in this list, not tile numbers, are split
@@ -86,8 +86,7 @@ __global__ void __launch_bounds__(128) flash_decode_kernel(const DecodeParams p)
         return r < rows ? p.q + ((size_t)(q_start + r / G) * p.Hq + hk * G + r % G) * D : nullptr;
     };
     rows_load_q(w, q_row);
-    w.pos[0] = g < rows ? first_pos + g / G : -1;
-    w.pos[1] = g + 8 < rows ? first_pos + (g + 8) / G : -1;
+    rows_place(w, g < rows ? first_pos + g / G : -1, g + 8 < rows ? first_pos + (g + 8) / G : -1, p.window);
     if (p.sink && split == 0 && warp == 0) {                           // once per row: the first warp of the first split
         w.m[0] = (g < rows ? p.sink[hk * G + g % G] : 0.f) * 1.4426950408889634f;
         w.m[1] = (g + 8 < rows ? p.sink[hk * G + (g + 8) % G] : 0.f) * 1.4426950408889634f;
@@ -119,8 +118,8 @@ __global__ void __launch_bounds__(128) flash_decode_kernel(const DecodeParams p)
             const int key0 = tl.tile(my_begin + i) * KT + warp * 16;
             if (key0 < kv_len)
                 rows_tile_auto<16>(w, smem + (2 * s) * TILE_ELEMS + warp * 16 * STRIDE,
-                                   smem + (2 * s + 1) * TILE_ELEMS + warp * 16 * STRIDE, key0, p.window, p.scale_log2,
-                                   first_pos, kv_len - 1, true, keep);
+                                   smem + (2 * s + 1) * TILE_ELEMS + warp * 16 * STRIDE, key0, lo_max, p.scale_log2,
+                                   first_pos, true, keep);
         }
         __syncthreads();
     }
@@ -305,7 +304,7 @@ __global__ void __launch_bounds__(128) flash_decode_cluster_kernel(const __grid_
     const int q_start = p.seg_q_start[seg], q_len = p.seg_q_len[seg], kv_len = p.seg_kv_len[seg];
     const int rows = min(q_len * G, 16);   // an item is one warp tile of 16 rows; rows beyond it are not this kernel's (see no_alloc.h)
     const int first_pos = kv_len - q_len;
-    const int key_lo = (p.window > 0 && first_pos - p.window + 1 > 0) ? first_pos - p.window + 1 : 0;
+    const int key_lo = first_seen_key(first_pos, p.window), lo_max = first_seen_key(kv_len - 1, p.window);
     const int tile_begin = key_lo / KT, tile_end = (kv_len + KT - 1) / KT;
     const int num_tiles = tile_end - tile_begin;
     // A stage holds KW key tiles, of which each warp takes 16 * KW keys; a split is a whole number of stages.
@@ -347,8 +346,7 @@ __global__ void __launch_bounds__(128) flash_decode_cluster_kernel(const __grid_
         return r < rows ? p.q + ((size_t)(q_start + r / G) * p.Hq + hk * G + r % G) * D : nullptr;
     };
     rows_load_q(w, q_row);
-    w.pos[0] = g < rows ? first_pos + g / G : -1;
-    w.pos[1] = g + 8 < rows ? first_pos + (g + 8) / G : -1;
+    rows_place(w, g < rows ? first_pos + g / G : -1, g + 8 < rows ? first_pos + (g + 8) / G : -1, p.window);
 
     for (int i = 0; i < n; ++i) {
         if (i + STAGES - 1 < n) load_stage(i + STAGES - 1);
@@ -359,8 +357,8 @@ __global__ void __launch_bounds__(128) flash_decode_cluster_kernel(const __grid_
         const bf16* ks = smem + (i % STAGES) * STAGE_ELEMS;
         const int key0 = (my_begin + i * KW) * KT + warp * NK;
         if (key0 < kv_len)
-            rows_tile_auto<NK>(w, ks + warp * NK * STRIDE, ks + KW * TILE_ELEMS + warp * NK * STRIDE, key0, p.window,
-                               p.scale_log2, first_pos, kv_len - 1, true);
+            rows_tile_auto<NK>(w, ks + warp * NK * STRIDE, ks + KW * TILE_ELEMS + warp * NK * STRIDE, key0, lo_max,
+                               p.scale_log2, first_pos, true);
         __syncthreads();
     }
     cp_async_wait<0>();
@@ -581,7 +579,7 @@ __global__ void __launch_bounds__(160) flash_decode_tma_kernel(const __grid_cons
     const int q_start = p.seg_q_start[seg], q_len = p.seg_q_len[seg], kv_len = p.seg_kv_len[seg];
     const int rows = min(q_len * G, 16);   // an item is one warp tile of 16 rows; rows beyond it are not this kernel's (see no_alloc.h)
     const int first_pos = kv_len - q_len;
-    const int key_lo = (p.window > 0 && first_pos - p.window + 1 > 0) ? first_pos - p.window + 1 : 0;
+    const int key_lo = first_seen_key(first_pos, p.window), lo_max = first_seen_key(kv_len - 1, p.window);
     // With kept first keys the list of key tiles is the kept ones, in whole stages of KW tiles, then the window's.  Where
     // the window's first tile lies among those stages the scan simply starts at tile 0.  Positions in the list are
     // shared out among the runs; a run's share is whole stages, so a stage never holds tiles of both parts.
@@ -766,8 +764,7 @@ __global__ void __launch_bounds__(160) flash_decode_tma_kernel(const __grid_cons
             return r < rows ? p.q + ((size_t)(q_start + r / G) * p.Hq + hk * G + r % G) * D : nullptr;
         };
         rows_load_q(w, q_row);
-        w.pos[0] = g < rows ? first_pos + g / G : -1;
-        w.pos[1] = g + 8 < rows ? first_pos + (g + 8) / G : -1;
+        rows_place(w, g < rows ? first_pos + g / G : -1, g + 8 < rows ? first_pos + (g + 8) / G : -1, p.window);
         if (p.sink && split == 0 && super == 0 && warp == 0) {             // once per row: the first warp of the first run
             w.m[0] = (g < rows ? p.sink[hk * G + g % G] : 0.f) * 1.4426950408889634f;
             w.m[1] = (g + 8 < rows ? p.sink[hk * G + (g + 8) % G] : 0.f) * 1.4426950408889634f;
@@ -800,7 +797,7 @@ __global__ void __launch_bounds__(160) flash_decode_tma_kernel(const __grid_cons
             }
             if (key0 < kv_len)
                 rows_tile_auto_in<NK>(w, SwizzledTile{base, HALF_BYTES}, SwizzledTile{base + KV_BYTES, HALF_BYTES}, key0,
-                                      p.window, p.scale_log2, first_pos, kv_len - 1, true, keep);
+                                      lo_max, p.scale_log2, first_pos, true, keep);
             __syncwarp();
             if (lane == 0) mbar_arrive(&sh.empty[s]);
         }
@@ -1070,6 +1067,7 @@ struct PrefillParams {
     // [Hq] or nullptr: with slopes, a score is cap tanh(scale q.k / cap) (cap 0: scale q.k) minus slopes[head] (p - j) for a key p - j back.
     const float* slopes = nullptr;
     float cap = 0.f, scale = 0.f;
+    int min_tiles;             // a unit has at least this many key tiles, unless its tile has fewer
 };
 
 __global__ void __launch_bounds__(128) flash_prefill_kernel(const PrefillParams p) {
@@ -1087,13 +1085,15 @@ __global__ void __launch_bounds__(128) flash_prefill_kernel(const PrefillParams 
     const int first_pos = kv_len - q_len;                    // position of the segment's first row
     const int tile_rows = min(64, q_len - row0);
     const int pos_first = first_pos + row0, pos_last = first_pos + row0 + tile_rows - 1;
-    const int key_lo = (p.window > 0 && pos_first - p.window + 1 > 0) ? pos_first - p.window + 1 : 0;
+    const int key_lo = first_seen_key(pos_first, p.window);
     const int tile_end = pos_last / KT + 1;
     const int keep = p.window > 0 ? p.keep : 0;
     const TileList tl(key_lo, tile_end, keep);                     // positions in this list, not tile numbers, are split
     const int num_tiles = tl.count;
-    const int per_split = (num_tiles + nsplit - 1) / nsplit;
-    const int n_valid = (num_tiles + per_split - 1) / per_split;   // units of this tile that have keys (a window may leave fewer)
+    // A window or chunks leave fewer key tiles than the host shared out: they are cut no finer than its units are.
+    const int parts = min(nsplit, (num_tiles + p.min_tiles - 1) / p.min_tiles);
+    const int per_split = (num_tiles + parts - 1) / parts;
+    const int n_valid = (num_tiles + per_split - 1) / per_split;   // units of this tile that have keys
     if (split >= n_valid) return;
     const int kt_begin = split * per_split;
     const int kt_end = min(num_tiles, kt_begin + per_split);
@@ -1109,11 +1109,10 @@ __global__ void __launch_bounds__(128) flash_prefill_kernel(const PrefillParams 
         return wrow0 + r < q_len ? p.q + ((size_t)(q_start + wrow0 + r) * p.Hq + h) * D : nullptr;
     };
     rows_load_q(w, q_row);
-    w.pos[0] = wrow0 + g < q_len ? first_pos + wrow0 + g : -1;
-    w.pos[1] = wrow0 + g + 8 < q_len ? first_pos + wrow0 + g + 8 : -1;
+    rows_place(w, wrow0 + g < q_len ? first_pos + wrow0 + g : -1, wrow0 + g + 8 < q_len ? first_pos + wrow0 + g + 8 : -1, p.window);
     const int warp_rows = min(16, q_len - wrow0);             // <= 0: the warp has no rows
     const int warp_pos_first = first_pos + wrow0, warp_pos_last = first_pos + wrow0 + warp_rows - 1;
-    const int warp_key_lo = (p.window > 0 && warp_pos_first - p.window + 1 > 0) ? warp_pos_first - p.window + 1 : 0;
+    const int warp_key_lo = first_seen_key(warp_pos_first, p.window), warp_lo_max = first_seen_key(warp_pos_last, p.window);
 
     constexpr int STAGES = PREFILL_STAGES;
 #pragma unroll
@@ -1133,8 +1132,8 @@ __global__ void __launch_bounds__(128) flash_prefill_kernel(const PrefillParams 
         const int s = i % STAGES;
         const int key0 = tl.tile(kt_begin + i) * KT;
         if (warp_rows > 0 && key0 <= warp_pos_last && (key0 + KT > warp_key_lo || key0 < keep))
-            rows_tile_auto<KT>(w, smem + (2 * s) * TILE_ELEMS, smem + (2 * s + 1) * TILE_ELEMS, key0, p.window, p.scale_log2,
-                               warp_pos_first, warp_pos_last, warp_rows == 16, keep);
+            rows_tile_auto<KT>(w, smem + (2 * s) * TILE_ELEMS, smem + (2 * s + 1) * TILE_ELEMS, key0, warp_lo_max, p.scale_log2,
+                               warp_pos_first, warp_rows == 16, keep);
         __syncthreads();
     }
     rows_finish_sum(w);
@@ -1223,9 +1222,9 @@ KVB_API int kvb_flash_prefill(const void* q, void* out, const void* k_pages, con
                               const int* block_table, int table_stride, const int* units, int n_units,
                               const int* seg_q_start, const int* seg_q_len, const int* seg_kv_len, float* scratch,
                               int* tickets, int Hq, int Hkv, int page_size, int window, float scale, const float* sink,
-                              int keep_first, const float* slopes, float cap, cudaStream_t stream) {
+                              int keep_first, const float* slopes, float cap, int min_tiles, cudaStream_t stream) {
     if (n_units <= 0) return KVB_OK;
-    if (Hkv < 1 || Hq % Hkv != 0) return KVB_ERR_SHAPE;
+    if (Hkv < 1 || Hq % Hkv != 0 || min_tiles < 1) return KVB_ERR_SHAPE;
     if (page_size < 1 || (page_size & (page_size - 1)) != 0) return KVB_ERR_SHAPE;
     if (Hq > 65535) return KVB_ERR_LIMIT;
     PrefillParams p;
@@ -1238,7 +1237,7 @@ KVB_API int kvb_flash_prefill(const void* q, void* out, const void* k_pages, con
     p.table_stride = table_stride; p.Hq = Hq; p.Hkv = Hkv; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window;
+    p.window = window; p.min_tiles = min_tiles;
     p.sink = sink; p.keep = keep_first;
     p.slopes = slopes; p.cap = cap; p.scale = scale;
     p.scale_log2 = scale * 1.4426950408889634f;

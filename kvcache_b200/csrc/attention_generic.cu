@@ -1,8 +1,8 @@
 // Causal attention over cache pages for any mix of rows, any head size and either storage
 // type: the kernel of the float32 path and the fallback of the bfloat16 one.
 //
-// One block per (row, query head).  The row's keys lo..pos (lo = 0, or pos - window + 1
-// for a windowed layer) are visited in chunks of the block's width: each thread scores
+// One block per (row, query head).  The row's keys lo..pos (lo = 0, pos - window + 1 for a
+// windowed layer, the first of the row's chunk for a negative `window`: first_seen_key) are visited in chunks of the block's width: each thread scores
 // one key, the block takes the chunk's maximum and sum, and threads then own output
 // dimensions for the weighted sum of values.  The running (max, sum, acc) update is the
 // reference's online softmax (src/qwen_kernels.cu:159-176: m' = max(m, s), c = e^{m-m'},
@@ -41,7 +41,7 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, const T*
     const int pos = positions[r];
     const int seg = row_segment[r];
     const int* table = block_table + (size_t)seg * table_stride;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = first_seen_key(pos, window);
     const int kept = min(keep_first, lo);          // keys before the window that stay visible
     const int visible = kept + pos - lo + 1;
     // Values as wide as the keys lie in a pool of their own; narrower ones (Dv < D) are the first Dv numbers of the key

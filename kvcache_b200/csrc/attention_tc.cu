@@ -11,7 +11,7 @@
 //   S = Q K^T   tcgen05.mma, M 128 x N 64 keys x K head size; Q and the key tile in 128-byte-swizzled shared
 //               memory (K-major), brought by TMA - the key tile page by page through the block table;
 //               S lands in tensor memory, 128 lanes x 64 columns.
-//   softmax     each thread reads its row of S with tcgen05.ld, masks it (causal limit, window), keeps the running
+//   softmax     each thread reads its row of S with tcgen05.ld, masks it (causal limit, window or chunk), keeps the running
 //               maximum and sum in base 2 (the reference's recurrence, src/qwen_kernels.cu:159-176), and writes
 //               P = 2^(s - m) as bfloat16 back into tensor memory (tcgen05.st), over the columns that held S.
 //   O_t = P V   tcgen05.mma, M 128 x N head size x K 64 keys; P is the A operand, read from tensor memory, the value
@@ -93,6 +93,7 @@ struct Params {
     // [Hq] or nullptr: with slopes, a score is cap tanh(scale q.k / cap) (cap 0: scale q.k) minus slopes[head] (p - j) for a key p - j back.
     const float* slopes;
     float cap, scale;
+    int min_tiles;             // a unit has at least this many key tiles, unless its tile has fewer
 };
 
 struct Shared {
@@ -148,7 +149,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int first_pos = kv_len - q_len;
     const int tile_rows = min(BQ, q_len - row0);
     const int pos_first = first_pos + row0, pos_last = pos_first + tile_rows - 1;
-    const int key_lo = (p.window > 0 && pos_first - p.window + 1 > 0) ? pos_first - p.window + 1 : 0;
+    const int key_lo = first_seen_key(pos_first, p.window);
     // The tile's key tiles are shared out among its units; a window may leave some units without any.
     // With kept first keys the list of key tiles is the kept tiles that lie wholly before the window's first tile, then
     // the window's; positions in that list, not tile numbers, are shared out.
@@ -157,7 +158,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int n_keep = min((keep + BKEYS - 1) / BKEYS, tile_begin);
     const int num_tiles = n_keep + tile_end - tile_begin;
     auto tile_at = [&](int i) -> int { return i < n_keep ? i : tile_begin - n_keep + i; };
-    const int per_split = (num_tiles + nsplit - 1) / nsplit;
+    // A window or chunks leave fewer key tiles than the host shared out: they are cut no finer than its units are.
+    const int parts = min(nsplit, (num_tiles + p.min_tiles - 1) / p.min_tiles);
+    const int per_split = (num_tiles + parts - 1) / parts;
     const int n_valid = (num_tiles + per_split - 1) / per_split;
     const int kt_begin = split * per_split, kt_end = min(num_tiles, kt_begin + per_split);
     const int n = kt_end - kt_begin;
@@ -267,6 +270,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         // ---- softmax warps: thread = row ----
         const int row = tid;                                    // 0..127 within the tile
         const int pos = row < tile_rows ? pos_first + row : -1;
+        const int lo = first_seen_key(pos, p.window);           // the first key the row sees
         const uint32_t lane_base = ((uint32_t)(warp * 32) << 16);
         float o[D];
 #pragma unroll
@@ -324,7 +328,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const int key0 = tile_at(kt_begin + i) * BKEYS;
             // Whether every row of this warp sees every key of the tile (then no element needs its mask).
-            const bool open = pos >= 0 && key0 + BKEYS - 1 <= pos && (p.window <= 0 || key0 > pos - p.window);
+            const bool open = pos >= 0 && key0 + BKEYS - 1 <= pos && key0 >= lo;
             const bool warp_open = __all_sync(0xffffffffu, open);
             // The row of S, read once.
             uint32_t sv[BKEYS];
@@ -348,7 +352,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 #pragma unroll
                 for (int e = 0; e < BKEYS; ++e) {
                     const int j = key0 + e;
-                    const bool seen = j <= pos && (p.window <= 0 || j > pos - p.window || j < keep);
+                    const bool seen = j <= pos && (j >= lo || j < keep);
                     if (!seen) sv[e] = __float_as_uint(NEG_INF);
                 }
             }
@@ -500,10 +504,10 @@ KVB_API int kvb_attention_tc(const void* q, void* out, const void* k_pages, cons
                              const int* block_table, int table_stride, const int* units, int n_units, float* scratch,
                              int* tickets, const int* seg_q_start, const int* seg_q_len, const int* seg_kv_len, int T,
                              int Hq, int Hkv, int page_size, int window, float scale, const float* sink, int keep_first,
-                             const float* slopes, float cap, int* err, cudaStream_t stream) {
+                             const float* slopes, float cap, int min_tiles, int* err, cudaStream_t stream) {
     using namespace atc;
     if (n_units <= 0) return KVB_OK;
-    if (Hkv < 1 || Hq % Hkv != 0 || Hq > 65535) return KVB_ERR_SHAPE;
+    if (Hkv < 1 || min_tiles < 1 || Hq % Hkv != 0 || Hq > 65535) return KVB_ERR_SHAPE;
     if (page_size < 8 || page_size > atc::BKEYS || (page_size & (page_size - 1)) != 0) return KVB_ERR_SHAPE;
     if (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) return KVB_ERR_ALIGN;
     CUtensorMap mq, mk, mv;
@@ -521,7 +525,7 @@ KVB_API int kvb_attention_tc(const void* q, void* out, const void* k_pages, cons
     p.seg_kv_len = seg_kv_len; p.table_stride = table_stride; p.Hq = Hq; p.Hkv = Hkv; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window;
+    p.window = window; p.min_tiles = min_tiles;
     p.sink = sink; p.keep = keep_first;
     p.slopes = slopes; p.cap = cap; p.scale = scale;
     p.scale_log2 = scale * 1.4426950408889634f;

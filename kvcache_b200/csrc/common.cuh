@@ -45,6 +45,14 @@ __device__ __forceinline__ float gated_pair(float g, float u, float limit) {
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
 }
 
+// Which keys up to its own a query at position `pos` sees, as one number `reach` (the `window` argument of the attention
+// kernels): w > 0 - the last w, so the first is max(0, pos - w + 1); -c < 0 - those of its chunk of c tokens, counted from the
+// request's first, so the first is pos - pos % c; 0 - all.  Returns the first.  It never decreases from one position to the next.
+__device__ __forceinline__ int first_seen_key(int pos, int reach) {
+    if (reach > 0) return max(0, pos - reach + 1);
+    return reach < 0 && pos > 0 ? pos - pos % -reach : 0;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

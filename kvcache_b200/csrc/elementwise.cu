@@ -1,4 +1,4 @@
-// Embedding gather, residual-add + RMSNorm, and the gated activation.
+// Embedding gather, residual-add + RMSNorm (or the norm that takes the mean off first), and the gated activation.
 //
 // What they replace in the reference: k_embed (src/qwen_kernels.cu:14-23),
 // k_rmsnorm with k_add in front of it (:26-43, :55-61) and k_silu_mul (:102-108).
@@ -53,12 +53,14 @@ KVB_API int kvb_embed(int dtype, const void* table, const int* ids, const int* s
 // One block per output row.
 //   rows == nullptr: r = blockIdx.x;  h[r] += delta[r] (if delta);  out[r] = norm(h[r]) * w
 //   rows != nullptr: r = rows[blockIdx.x]; v = h[r] + delta[r]; out[blockIdx.x] = norm(v) * w; h untouched
-// `ds` (float32 [H], or null): delta is multiplied by it, channel by channel, before the add (a layer's output scale).
+// `ds` (float32 [H], or null): delta is multiplied by it, channel by channel, before the add (a layer's output scale); `db`
+// (float32 [H], or null): first this is added to delta (the bias of the product that made it): h += (delta + db) * ds.
 // norm(v) = v * rsqrt(mean(v^2) + eps), everything in float32 (src/qwen_kernels.cu:26-40:
-// fp32 sum of squares, (x * inv) * w, one rounding at the store).
-template <typename T>
+// fp32 sum of squares, (x * inv) * w, one rounding at the store).  CENTRED: norm(v) = d * rsqrt(mean(d^2) + eps) with
+// d = v - mean(v); the mean is taken first and the squares are those of the deviations.
+template <typename T, bool CENTRED>
 __global__ void add_rmsnorm_kernel(float* __restrict__ h, const T* __restrict__ delta, const float* __restrict__ ds,
-                                   const float* __restrict__ w, T* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
+                                   const float* __restrict__ db, const float* __restrict__ w, T* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
     pdl_wait();
     pdl_launch_dependents();
     __shared__ float scratch[33];
@@ -66,20 +68,34 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ h, const T* __restrict__ 
     const int r = rows ? rows[o] : o;
     float* hr = h + (size_t)r * H;
     const T* dr = delta ? delta + (size_t)r * H : nullptr;
+    auto step = [&](int i) {
+        const float d = to_f32<T>(dr[i]) + (db ? db[i] : 0.f);
+        return ds ? d * ds[i] : d;
+    };
     float ss = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = hr[i];
-        if (dr) v += ds ? to_f32<T>(dr[i]) * ds[i] : to_f32<T>(dr[i]);
+        if (dr) v += step(i);
         if (!rows && dr) hr[i] = v;
-        ss += v * v;
+        ss += CENTRED ? v : v * v;
     }
-    const float total = block_sum(ss, scratch);
+    float total = block_sum(ss, scratch), mean = 0.f;
+    if (CENTRED) {
+        mean = total / (float)H;
+        ss = 0.f;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            float v = hr[i];
+            if (rows && dr) v += step(i);
+            ss += (v - mean) * (v - mean);
+        }
+        total = block_sum(ss, scratch);
+    }
     const float inv = 1.f / sqrtf(total / (float)H + eps);
     T* orow = out + (size_t)o * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = hr[i];
-        if (rows && dr) v += ds ? to_f32<T>(dr[i]) * ds[i] : to_f32<T>(dr[i]);
-        orow[i] = from_f32<T>(v * inv * w[i]);
+        if (rows && dr) v += step(i);
+        orow[i] = from_f32<T>((v - mean) * inv * w[i]);
     }
 }
 
@@ -109,8 +125,22 @@ template <> struct Vec4<bf16> {
 // the sum of squares and the scaling, and reads the norm's weight - which no kernel writes - before it waits
 // for the kernel that makes `delta`; rows longer than KEEP * 4 * blockDim are read a second time.
 template <typename T>
+__device__ __forceinline__ float4 delta_step(const T* dr, const float* ds, const float* db, int i) {
+    float4 d = Vec4<T>::load(dr + i);
+    if (db) {
+        const float4 c = *reinterpret_cast<const float4*>(db + i);
+        d.x += c.x; d.y += c.y; d.z += c.z; d.w += c.w;
+    }
+    if (ds) {
+        const float4 c = *reinterpret_cast<const float4*>(ds + i);
+        d.x *= c.x; d.y *= c.y; d.z *= c.z; d.w *= c.w;
+    }
+    return d;
+}
+
+template <typename T, bool CENTRED>
 __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const T* __restrict__ delta, const float* __restrict__ ds,
-                                       const float* __restrict__ w, T* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
+                                       const float* __restrict__ db, const float* __restrict__ w, T* __restrict__ out, const int* __restrict__ rows, int H, float eps) {
     constexpr int KEEP = 2;
     __shared__ float scratch[33];
     const int o = blockIdx.x;
@@ -130,11 +160,7 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const T* __restric
     auto fetch = [&](int i) {
         float4 v = *reinterpret_cast<const float4*>(hr + i);
         if (dr) {
-            float4 d = Vec4<T>::load(dr + i);
-            if (ds) {
-                const float4 c = *reinterpret_cast<const float4*>(ds + i);
-                d.x *= c.x; d.y *= c.y; d.z *= c.z; d.w *= c.w;
-            }
+            const float4 d = delta_step(dr, ds, db, i);
             v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
         }
         return v;
@@ -142,21 +168,44 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const T* __restric
     auto square = [&](const float4& v) {                   // summed element by element, as the scalar kernel's thread does
         ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w;
     };
+    auto first = [&](const float4& v) {                    // what the first sum is over
+        if (CENTRED) { ss += v.x; ss += v.y; ss += v.z; ss += v.w; }
+        else square(v);
+    };
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
         const int i = (threadIdx.x + k * blockDim.x) * 4;
         if (i < H) {
             kept[k] = fetch(i);
             if (dr && !rows) *reinterpret_cast<float4*>(hr + i) = kept[k];
-            square(kept[k]);
+            first(kept[k]);
         }
     }
     for (int i = (threadIdx.x + KEEP * blockDim.x) * 4; i < H; i += blockDim.x * 4) {
         const float4 v = fetch(i);
         if (dr && !rows) *reinterpret_cast<float4*>(hr + i) = v;
-        square(v);
+        first(v);
     }
-    const float total = block_sum(ss, scratch);
+    float total = block_sum(ss, scratch);
+    float mean = 0.f;
+    if (CENTRED) {
+        mean = total / (float)H;
+        ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = (threadIdx.x + k * blockDim.x) * 4;
+            if (i < H) {
+                kept[k].x -= mean; kept[k].y -= mean; kept[k].z -= mean; kept[k].w -= mean;
+                square(kept[k]);
+            }
+        }
+        for (int i = (threadIdx.x + KEEP * blockDim.x) * 4; i < H; i += blockDim.x * 4) {
+            float4 v = rows ? fetch(i) : *reinterpret_cast<const float4*>(hr + i);
+            v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean;
+            square(v);
+        }
+        total = block_sum(ss, scratch);
+    }
     const float inv = 1.f / sqrtf(total / (float)H + eps);
     T* orow = out + (size_t)o * H;
 #pragma unroll
@@ -169,15 +218,8 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const T* __restric
     }
     for (int i = (threadIdx.x + KEEP * blockDim.x) * 4; i < H; i += blockDim.x * 4) {
         // Beyond what the registers keep: read again (after an in-place update the row already holds the sum).
-        float4 v = *reinterpret_cast<const float4*>(hr + i);
-        if (rows && dr) {
-            float4 d = Vec4<T>::load(dr + i);
-            if (ds) {
-                const float4 c = *reinterpret_cast<const float4*>(ds + i);
-                d.x *= c.x; d.y *= c.y; d.z *= c.z; d.w *= c.w;
-            }
-            v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
-        }
+        float4 v = rows ? fetch(i) : *reinterpret_cast<const float4*>(hr + i);
+        if (CENTRED) { v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean; }
         const float4 g = *reinterpret_cast<const float4*>(w + i);
         Vec4<T>::store(orow + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
     }
@@ -188,9 +230,9 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ h, const T* __restric
 // above in the same order - lane l's chunk c is thread l + 32 c's chunk there, each group of 32 is summed by the same
 // shuffles, and the groups are added one after the other - so a row's result is bit for bit the same whichever of
 // the two kernels a step's row count selects.  Needs H <= 128 C.
-template <typename T, int C>
+template <typename T, int C, bool CENTRED>
 __global__ void add_rmsnorm_warp_kernel(float* __restrict__ h, const T* __restrict__ delta, const float* __restrict__ ds,
-                                        const float* __restrict__ w, T* __restrict__ out, const int* __restrict__ rows, int n_out, int H,
+                                        const float* __restrict__ db, const float* __restrict__ w, T* __restrict__ out, const int* __restrict__ rows, int n_out, int H,
                                         float eps) {
     const int lane = threadIdx.x & 31;
     const int o = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -217,11 +259,7 @@ __global__ void add_rmsnorm_warp_kernel(float* __restrict__ h, const T* __restri
         for (int c = 0; c < C; ++c) {
             const int i = (lane + 32 * c) * 4;
             if (i < H) {
-                float4 d = Vec4<T>::load(dr + i);
-                if (ds) {
-                    const float4 e = *reinterpret_cast<const float4*>(ds + i);
-                    d.x *= e.x; d.y *= e.y; d.z *= e.z; d.w *= e.w;
-                }
+                const float4 d = delta_step(dr, ds, db, i);
                 kept[c].x += d.x; kept[c].y += d.y; kept[c].z += d.z; kept[c].w += d.w;
                 if (!rows) *reinterpret_cast<float4*>(hr + i) = kept[c];
             }
@@ -229,6 +267,20 @@ __global__ void add_rmsnorm_warp_kernel(float* __restrict__ h, const T* __restri
     }
     const int groups = (H / 4 + 31) >> 5;                   // the warps that the kernel above would run
     float total = 0.f;
+    if (CENTRED) {
+        float mean = 0.f;
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            float s = 0.f;
+            s += kept[c].x; s += kept[c].y; s += kept[c].z; s += kept[c].w;
+            s = warp_sum(s);
+            if (c < groups) mean += s;
+        }
+        mean /= (float)H;
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+            if ((lane + 32 * c) * 4 < H) { kept[c].x -= mean; kept[c].y -= mean; kept[c].z -= mean; kept[c].w -= mean; }
+    }
 #pragma unroll
     for (int c = 0; c < C; ++c) {
         float ss = 0.f;
@@ -248,49 +300,48 @@ __global__ void add_rmsnorm_warp_kernel(float* __restrict__ h, const T* __restri
     }
 }
 
-template <typename T>
-static bool launch_rmsnorm_warp(float* h, const T* delta, const float* ds, const float* w, T* out, const int* rows, int n_out, int H,
+template <typename T, bool CENTRED>
+static bool launch_rmsnorm_warp(float* h, const T* delta, const float* ds, const float* db, const float* w, T* out, const int* rows, int n_out, int H,
                                 float eps, cudaStream_t stream) {
     constexpr int WARPS = 2;
     const dim3 grid((n_out + WARPS - 1) / WARPS), block(32 * WARPS);
-    if (H <= 512) kvb_launch(add_rmsnorm_warp_kernel<T, 4>, grid, block, 0, stream, h, delta, ds, w, out, rows, n_out, H, eps);
-    else if (H <= 1024) kvb_launch(add_rmsnorm_warp_kernel<T, 8>, grid, block, 0, stream, h, delta, ds, w, out, rows, n_out, H, eps);
-    else if (H <= 1536) kvb_launch(add_rmsnorm_warp_kernel<T, 12>, grid, block, 0, stream, h, delta, ds, w, out, rows, n_out, H, eps);
-    else if (H <= 2048) kvb_launch(add_rmsnorm_warp_kernel<T, 16>, grid, block, 0, stream, h, delta, ds, w, out, rows, n_out, H, eps);
+    if (H <= 512) kvb_launch(add_rmsnorm_warp_kernel<T, 4, CENTRED>, grid, block, 0, stream, h, delta, ds, db, w, out, rows, n_out, H, eps);
+    else if (H <= 1024) kvb_launch(add_rmsnorm_warp_kernel<T, 8, CENTRED>, grid, block, 0, stream, h, delta, ds, db, w, out, rows, n_out, H, eps);
+    else if (H <= 1536) kvb_launch(add_rmsnorm_warp_kernel<T, 12, CENTRED>, grid, block, 0, stream, h, delta, ds, db, w, out, rows, n_out, H, eps);
+    else if (H <= 2048) kvb_launch(add_rmsnorm_warp_kernel<T, 16, CENTRED>, grid, block, 0, stream, h, delta, ds, db, w, out, rows, n_out, H, eps);
     else return false;
     return true;
 }
 
 constexpr int RMSNORM_WARP_MIN_ROWS = 256;                  // below this a block per row has more loads in flight
 
-KVB_API int kvb_add_rmsnorm(int dtype, float* h, const void* delta, const float* ds, const float* w, void* out, const int* rows,
-                            int n_out, int H, float eps, cudaStream_t stream) {
-    if (n_out <= 0) return KVB_OK;
-    const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
-    const bool vec = H % 4 == 0 && ((((uintptr_t)h | (uintptr_t)w | (uintptr_t)out | (uintptr_t)delta | (uintptr_t)ds) & 15) == 0);
-    // One chunk of four per thread where the row allows it.
-    const int vec_threads = H / 4 >= 1024 ? 1024 : (H / 4 + 31) / 32 * 32;
-    if (vec && n_out >= RMSNORM_WARP_MIN_ROWS) {
-        if (dtype == KVB_F32 && launch_rmsnorm_warp<float>(h, (const float*)delta, ds, w, (float*)out, rows, n_out, H, eps, stream))
-            return kvb_launch_status();
-        if (dtype == KVB_BF16 && launch_rmsnorm_warp<bf16>(h, (const bf16*)delta, ds, w, (bf16*)out, rows, n_out, H, eps, stream))
-            return kvb_launch_status();
-    }
-    if (vec && dtype == KVB_F32) {
-        kvb_launch(add_rmsnorm_vec_kernel<float>, dim3(n_out), dim3(vec_threads), 0, stream, h, (const float*)delta, ds, w, (float*)out, rows, H, eps);
+template <typename T, bool CENTRED>
+static int launch_add_norm(float* h, const T* delta, const float* ds, const float* db, const float* w, T* out, const int* rows, int n_out,
+                           int H, float eps, cudaStream_t stream) {
+    const bool vec = H % 4 == 0 && ((((uintptr_t)h | (uintptr_t)w | (uintptr_t)out | (uintptr_t)delta | (uintptr_t)ds | (uintptr_t)db) & 15) == 0);
+    if (vec && n_out >= RMSNORM_WARP_MIN_ROWS && launch_rmsnorm_warp<T, CENTRED>(h, delta, ds, db, w, out, rows, n_out, H, eps, stream))
         return kvb_launch_status();
+    if (vec) {      // one chunk of four per thread where the row allows it
+        const int threads = H / 4 >= 1024 ? 1024 : (H / 4 + 31) / 32 * 32;
+        kvb_launch(add_rmsnorm_vec_kernel<T, CENTRED>, dim3(n_out), dim3(threads), 0, stream, h, delta, ds, db, w, out, rows, H, eps);
+    } else {
+        const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
+        kvb_launch(add_rmsnorm_kernel<T, CENTRED>, dim3(n_out), dim3(threads), 0, stream, h, delta, ds, db, w, out, rows, H, eps);
     }
-    if (vec && dtype == KVB_BF16) {
-        kvb_launch(add_rmsnorm_vec_kernel<bf16>, dim3(n_out), dim3(vec_threads), 0, stream, h, (const bf16*)delta, ds, w, (bf16*)out, rows, H, eps);
-        return kvb_launch_status();
-    }
-    if (dtype == KVB_F32)
-        kvb_launch(add_rmsnorm_kernel<float>, dim3(n_out), dim3(threads), 0, stream, h, (const float*)delta, ds, w, (float*)out, rows, H, eps);
-    else if (dtype == KVB_BF16)
-        kvb_launch(add_rmsnorm_kernel<bf16>, dim3(n_out), dim3(threads), 0, stream, h, (const bf16*)delta, ds, w, (bf16*)out, rows, H, eps);
-    else
-        return KVB_ERR_DTYPE;
     return kvb_launch_status();
+}
+
+// `centred` 1: the mean is taken off before the norm divides (see add_rmsnorm_kernel).
+KVB_API int kvb_add_norm(int dtype, int centred, float* h, const void* delta, const float* ds, const float* db, const float* w, void* out,
+                         const int* rows, int n_out, int H, float eps, cudaStream_t stream) {
+    if (n_out <= 0) return KVB_OK;
+    if (dtype == KVB_F32)
+        return centred ? launch_add_norm<float, true>(h, (const float*)delta, ds, db, w, (float*)out, rows, n_out, H, eps, stream)
+                       : launch_add_norm<float, false>(h, (const float*)delta, ds, db, w, (float*)out, rows, n_out, H, eps, stream);
+    if (dtype == KVB_BF16)
+        return centred ? launch_add_norm<bf16, true>(h, (const bf16*)delta, ds, db, w, (bf16*)out, rows, n_out, H, eps, stream)
+                       : launch_add_norm<bf16, false>(h, (const bf16*)delta, ds, db, w, (bf16*)out, rows, n_out, H, eps, stream);
+    return KVB_ERR_DTYPE;
 }
 
 // out[r, i] = silu(gate[r, i]) * up[r, i],  silu(g) = g / (1 + exp(-g))   (src/qwen_kernels.cu:102-105).

@@ -98,6 +98,7 @@ struct WarpRows {
     float o[NT_O][4];      // output accumulators: [.][0..1] row g, [.][2..3] row g + 8
     float m[2], l[2];      // running maximum (base-2 units) and this thread's share of the running sum
     int pos[2];            // absolute position of rows g and g + 8 (-1: the row does not exist)
+    int lo[2];             // the first key each of the two sees (see first_seen_key)
     // Scores that are more than scale * q.k (see rows_bias): s = cap tanh(scale q.k / cap) - slope (p - j).
     bool biased;
     float scale, cap, slope[2];
@@ -108,8 +109,18 @@ __device__ __forceinline__ void rows_init(WarpRows& w) {
     for (int i = 0; i < NT_O; ++i) w.o[i][0] = w.o[i][1] = w.o[i][2] = w.o[i][3] = 0.f;
     w.m[0] = w.m[1] = NEG_INF;
     w.l[0] = w.l[1] = 0.f;
+    w.pos[0] = w.pos[1] = -1;
+    w.lo[0] = w.lo[1] = 0;
     w.biased = false;
     w.scale = w.cap = w.slope[0] = w.slope[1] = 0.f;
+}
+
+// The rows' positions and what they see under `reach` (the kernels' `window` argument).
+__device__ __forceinline__ void rows_place(WarpRows& w, int pos0, int pos1, int reach) {
+    w.pos[0] = pos0;
+    w.pos[1] = pos1;
+    w.lo[0] = first_seen_key(pos0, reach);
+    w.lo[1] = first_seen_key(pos1, reach);
 }
 
 // From now on the rows' scores are s = cap * tanh(scale * q.k / cap) (cap 0: scale * q.k) minus slope * (p - j) for a key
@@ -181,11 +192,12 @@ struct SwizzledTile {          // as TMA leaves it with the 128-byte swizzle: ro
 
 // NK keys [key0, key0 + NK) whose rows start at row 0 of `kt` / `vt`: scores, masking, running
 // softmax, weighted sum.  NK is a multiple of 16 (a whole tile, or a part of one).
-// A key j is seen by a row at position p iff key_lo(p) <= j <= p, key_lo(p) = max(0, p - window + 1), or j < keep and j <= p.
+// A key j is seen by a row at position p iff lo(p) <= j <= p, lo(p) the first key of its window or chunk (rows_place), or
+// j < keep and j <= p.
 // MASKED = false: the caller knows that every row sees every key of the range.
 template <int NK, bool MASKED, class Tile>
-__device__ __forceinline__ void rows_tile(WarpRows& w, const Tile& kt, const Tile& vt, int key0, int window,
-                                          float scale_log2, int keep = 0) {
+__device__ __forceinline__ void rows_tile(WarpRows& w, const Tile& kt, const Tile& vt, int key0, float scale_log2,
+                                          int keep = 0) {
     const int lane = threadIdx.x & 31, t = lane & 3;
     float s[NK / 8][4];
 #pragma unroll
@@ -227,7 +239,7 @@ __device__ __forceinline__ void rows_tile(WarpRows& w, const Tile& kt, const Til
             if (MASKED) {
                 const int j = key0 + n * 8 + 2 * t + (e & 1);
                 const int p = w.pos[e >> 1];
-                const bool seen = j <= p && (window <= 0 || j > p - window || j < keep);
+                const bool seen = j <= p && (j >= w.lo[e >> 1] || j < keep);
                 if (!seen) s[n][e] = NEG_INF;
             }
             mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
@@ -280,19 +292,19 @@ __device__ __forceinline__ void rows_tile(WarpRows& w, const Tile& kt, const Til
     }
 }
 
-// NK keys from key0 on: masked only if a row may miss one of them.  `pos_min` / `pos_max`: smallest and
-// largest position among the warp's existing rows.
+// NK keys from key0 on: masked only if a row may miss one of them.  `pos_min`: smallest position among the warp's
+// existing rows; `lo_max`: the first key that the row with the largest one sees.
 template <int NK, class Tile>
-__device__ __forceinline__ void rows_tile_auto_in(WarpRows& w, const Tile& kt, const Tile& vt, int key0, int window,
-                                               float scale_log2, int pos_min, int pos_max, bool all_rows_exist, int keep = 0) {
-    const bool open = all_rows_exist && key0 + NK - 1 <= pos_min && (window <= 0 || key0 > pos_max - window);
-    if (open) rows_tile<NK, false>(w, kt, vt, key0, window, scale_log2);
-    else rows_tile<NK, true>(w, kt, vt, key0, window, scale_log2, keep);
+__device__ __forceinline__ void rows_tile_auto_in(WarpRows& w, const Tile& kt, const Tile& vt, int key0, int lo_max,
+                                               float scale_log2, int pos_min, bool all_rows_exist, int keep = 0) {
+    const bool open = all_rows_exist && key0 + NK - 1 <= pos_min && key0 >= lo_max;
+    if (open) rows_tile<NK, false>(w, kt, vt, key0, scale_log2);
+    else rows_tile<NK, true>(w, kt, vt, key0, scale_log2, keep);
 }
 template <int NK>
-__device__ __forceinline__ void rows_tile_auto(WarpRows& w, const bf16* ks, const bf16* vs, int key0, int window,
-                                               float scale_log2, int pos_min, int pos_max, bool all_rows_exist, int keep = 0) {
-    rows_tile_auto_in<NK>(w, PaddedTile{ks}, PaddedTile{vs}, key0, window, scale_log2, pos_min, pos_max, all_rows_exist, keep);
+__device__ __forceinline__ void rows_tile_auto(WarpRows& w, const bf16* ks, const bf16* vs, int key0, int lo_max,
+                                               float scale_log2, int pos_min, bool all_rows_exist, int keep = 0) {
+    rows_tile_auto_in<NK>(w, PaddedTile{ks}, PaddedTile{vs}, key0, lo_max, scale_log2, pos_min, all_rows_exist, keep);
 }
 
 // Sums each row's l over the four threads that share it.

@@ -19,7 +19,8 @@
 // and the block still waits (bounded) for the copies it issued, frees its tensor memory and returns.
 //
 // Gated output (`swiglu`): W holds gate and up rows interleaved in eights (see gemm_skinny.cu);
-// the epilogue writes silu(gate) * up to out[M, N / 2] (src/qwen_kernels.cu:102-105).
+// the epilogue writes silu(gate) * up to out[M, N / 2] (src/qwen_kernels.cu:102-105), or, with a `limit` above 0, the clamped
+// gated activation (gated_pair in common.cuh).
 #include "tc_common.cuh"
 
 namespace tc {
@@ -36,7 +37,7 @@ constexpr int PAIR_STAGES = 6 / PAIR_KSUB;
 // conversion, or the gated activation on interleaved gate/up columns.
 template <typename TOut, bool SWIGLU>
 __device__ __forceinline__ void store_chunk(const uint32_t* r, const float* __restrict__ bias, TOut* __restrict__ y, int m,
-                                            int n, int N) {
+                                            int n, int N, float limit) {
     if (SWIGLU) {
         // columns n .. n+7 gate, n+8 .. n+15 up, twice per 32: 16 outputs at column n / 2
         TOut* out = y + (size_t)m * (N >> 1) + (n >> 1);
@@ -45,8 +46,14 @@ __device__ __forceinline__ void store_chunk(const uint32_t* r, const float* __re
         for (int blk = 0; blk < 2; ++blk)
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-                const float gate = __uint_as_float(r[16 * blk + i]), up = __uint_as_float(r[16 * blk + 8 + i]);
-                v[8 * blk + i] = __fdividef(gate, 1.f + __expf(-gate)) * up;
+                float gate = __uint_as_float(r[16 * blk + i]), up = __uint_as_float(r[16 * blk + 8 + i]);
+                if (limit > 0.f) {                  // the same for every thread of the launch
+                    gate = fminf(gate, limit);
+                    up = fminf(fmaxf(up, -limit), limit);
+                    v[8 * blk + i] = __fdividef(gate, 1.f + __expf(-1.702f * gate)) * (up + 1.f);
+                } else {
+                    v[8 * blk + i] = __fdividef(gate, 1.f + __expf(-gate)) * up;
+                }
             }
         if (n + 32 <= N && sizeof(TOut) == 2 && (N & 15) == 0) {
             uint32_t packed[8];
@@ -101,7 +108,7 @@ struct Shared {
 template <int BN, typename TOut, bool SWIGLU>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                    const float* __restrict__ bias, TOut* __restrict__ y, int M, int N, int K, int* __restrict__ err) {
+                    const float* __restrict__ bias, TOut* __restrict__ y, int M, int N, int K, float limit, int* __restrict__ err) {
     constexpr int B_BYTES = BN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
     constexpr int STAGES = BN == 256 ? 4 : 6;
     extern __shared__ unsigned char smem_raw[];
@@ -190,7 +197,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                 tmem_ld32(tmem + ((uint32_t)(quarter * 32) << 16) + b * BN + c * 32, r);
                 const int n = n0 + c * 32;
                 if (m >= M || n >= N) continue;
-                store_chunk<TOut, SWIGLU>(r, bias, y, m, n, N);
+                store_chunk<TOut, SWIGLU>(r, bias, y, m, n, N, limit);
             }
             // This warp has read its part of the accumulator: hand it back to the MMA warp.
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -257,7 +264,7 @@ __device__ __forceinline__ void mbar_arrive_leader(uint64_t* bar) {
 template <int BN, typename TOut, bool SWIGLU>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                         const float* __restrict__ bias, TOut* __restrict__ y, int M, int N, int K, int* __restrict__ err) {
+                         const float* __restrict__ bias, TOut* __restrict__ y, int M, int N, int K, float limit, int* __restrict__ err) {
     // BN columns of y a tile, 256 or a little fewer: the launcher takes the width whose last round of tiles wastes least.
     static_assert(BN % 32 == 0 && BN >= 128 && BN <= 256, "tile width");
     constexpr int HALF_N = BN / 2, ACC_STRIDE = 256;             // the two accumulators lie 256 columns apart whatever BN
@@ -374,7 +381,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
                 tmem_ld32(tmem + ((uint32_t)(quarter * 32) << 16) + b * ACC_STRIDE + c * 32, r);
                 const int n = n0 + c * 32;
                 if (m >= M || n >= N) continue;
-                store_chunk<TOut, SWIGLU>(r, bias, y, m, n, N);
+                store_chunk<TOut, SWIGLU>(r, bias, y, m, n, N, limit);
             }
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
             __syncwarp();
@@ -431,7 +438,7 @@ static int sm_count() {
 }
 
 template <int BN, typename TOut, bool SWIGLU>
-static int launch(const void* x, const void* w, const float* bias, TOut* y, int M, int N, int K, int* err, cudaStream_t stream) {
+static int launch(const void* x, const void* w, const float* bias, TOut* y, int M, int N, int K, float limit, int* err, cudaStream_t stream) {
     CUtensorMap mx, mw;
     int rc = make_map(&mx, x, M, K, BM);
     if (rc != KVB_OK) return rc;
@@ -448,12 +455,12 @@ static int launch(const void* x, const void* w, const float* bias, TOut* y, int 
     }
     const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
     const int blocks = tiles < sm_count() ? tiles : sm_count();
-    kernel<<<blocks, THREADS, smem, stream>>>(mx, mw, bias, y, M, N, K, err);
+    kernel<<<blocks, THREADS, smem, stream>>>(mx, mw, bias, y, M, N, K, limit, err);
     return kvb_launch_status();
 }
 
 template <int BN, typename TOut, bool SWIGLU>
-static int launch_pair(const void* x, const void* w, const float* bias, TOut* y, int M, int N, int K, int* err, cudaStream_t stream) {
+static int launch_pair(const void* x, const void* w, const float* bias, TOut* y, int M, int N, int K, float limit, int* err, cudaStream_t stream) {
     CUtensorMap mx, mw;
     int rc = make_map(&mx, x, M, K, BM);
     if (rc != KVB_OK) return rc;
@@ -470,14 +477,14 @@ static int launch_pair(const void* x, const void* w, const float* bias, TOut* y,
     const int tiles = ((M + 2 * BM - 1) / (2 * BM)) * ((N + BN - 1) / BN);
     int pairs = sm_count() / 2;
     if (tiles < pairs) pairs = tiles;
-    kvb_launch(kernel, dim3(2 * pairs), dim3(THREADS), smem, stream, mx, mw, bias, y, M, N, K, err);   // the cluster of two is the kernel's own attribute
+    kvb_launch(kernel, dim3(2 * pairs), dim3(THREADS), smem, stream, mx, mw, bias, y, M, N, K, limit, err);   // the cluster of two is the kernel's own attribute
     return kvb_launch_status();
 }
 
 // Two SMs on a 256 x 256 tile where there are enough such tiles; else 256-wide tiles on one SM (they halve the
 // shared-memory traffic per product, but only pay when there are enough of them); else 128-wide tiles.
 template <typename TOut, bool SWIGLU>
-static int dispatch(const void* x, const void* w, const float* bias, TOut* y, int M, int N, int K, int* err, cudaStream_t stream) {
+static int dispatch(const void* x, const void* w, const float* bias, TOut* y, int M, int N, int K, float limit, int* err, cudaStream_t stream) {
     const int wide_tiles = ((M + BM - 1) / BM) * ((N + 255) / 256);
     const int pair_tiles = ((M + 2 * BM - 1) / (2 * BM)) * ((N + 255) / 256);
     if (pair_mode() && pair_tiles >= sm_count()) {
@@ -489,12 +496,12 @@ static int dispatch(const void* x, const void* w, const float* bias, TOut* y, in
         // A narrower tile reads more operand bytes per product, so it must save a twentieth at least (4,096 x 17,920 x
         // 1,536: 18 rounds of 224 against 16 of 256 are 1.6 % less by this count and measured 2.5 % more time).
         const long long wide = cost(256) * 20, c224 = cost(224) * 21, c192 = cost(192) * 21;
-        if (c224 < wide && c224 <= c192) return launch_pair<224, TOut, SWIGLU>(x, w, bias, y, M, N, K, err, stream);
-        if (c192 < wide) return launch_pair<192, TOut, SWIGLU>(x, w, bias, y, M, N, K, err, stream);
-        return launch_pair<256, TOut, SWIGLU>(x, w, bias, y, M, N, K, err, stream);
+        if (c224 < wide && c224 <= c192) return launch_pair<224, TOut, SWIGLU>(x, w, bias, y, M, N, K, limit, err, stream);
+        if (c192 < wide) return launch_pair<192, TOut, SWIGLU>(x, w, bias, y, M, N, K, limit, err, stream);
+        return launch_pair<256, TOut, SWIGLU>(x, w, bias, y, M, N, K, limit, err, stream);
     }
-    if (wide_tiles >= sm_count()) return launch<256, TOut, SWIGLU>(x, w, bias, y, M, N, K, err, stream);
-    return launch<128, TOut, SWIGLU>(x, w, bias, y, M, N, K, err, stream);
+    if (wide_tiles >= sm_count()) return launch<256, TOut, SWIGLU>(x, w, bias, y, M, N, K, limit, err, stream);
+    return launch<128, TOut, SWIGLU>(x, w, bias, y, M, N, K, limit, err, stream);
 }
 
 }  // namespace tc
@@ -502,17 +509,18 @@ static int dispatch(const void* x, const void* w, const float* bias, TOut* y, in
 // x [M, K], w [N, K] bfloat16 row-major; bias float32 [N] or null; y [M, N] bfloat16 (out_dtype 1) or float32 (0),
 // or with swiglu = 1 [M, N / 2] from interleaved gate/up rows (N % 16 == 0, no bias).
 // Refuses K % 8 != 0 and operands that are not 16-byte aligned.
+// With swiglu = 1, `limit` above 0 is the clamped gated activation's constant (0: silu(gate) * up).
 KVB_API int kvb_gemm_tcgen05(int out_dtype, int swiglu, const void* x, const void* w, const float* bias, void* y, int M,
-                             int N, int K, int* err, cudaStream_t stream) {
+                             int N, int K, float limit, int* err, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return KVB_OK;
     if (K <= 0 || K % 8 != 0) return KVB_ERR_SHAPE;
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)y) & 15) return KVB_ERR_ALIGN;
     if (swiglu && (N % 16 != 0 || bias != nullptr)) return KVB_ERR_SHAPE;
     if (out_dtype == KVB_BF16)
-        return swiglu ? tc::dispatch<bf16, true>(x, w, bias, (bf16*)y, M, N, K, err, stream)
-                      : tc::dispatch<bf16, false>(x, w, bias, (bf16*)y, M, N, K, err, stream);
+        return swiglu ? tc::dispatch<bf16, true>(x, w, bias, (bf16*)y, M, N, K, limit, err, stream)
+                      : tc::dispatch<bf16, false>(x, w, bias, (bf16*)y, M, N, K, limit, err, stream);
     if (out_dtype == KVB_F32)
-        return swiglu ? tc::dispatch<float, true>(x, w, bias, (float*)y, M, N, K, err, stream)
-                      : tc::dispatch<float, false>(x, w, bias, (float*)y, M, N, K, err, stream);
+        return swiglu ? tc::dispatch<float, true>(x, w, bias, (float*)y, M, N, K, limit, err, stream)
+                      : tc::dispatch<float, false>(x, w, bias, (float*)y, M, N, K, limit, err, stream);
     return KVB_ERR_DTYPE;
 }

@@ -2,10 +2,13 @@
 //
 //   route_top      per row: the `top` experts with the largest float32 logits, weights = softmax over those logits only,
 //                  or the softmax over all experts' logits at the chosen ones, as they are
+//   route_sigmoid  per row: scores s = sigmoid(logits); the choice by s + correction, within the best groups of experts;
+//                  weights = scale * s / (sum of the chosen s + 1e-20)
 //   routed_plan    (row, choice) pairs sorted by expert: where each pair sits, and the list of row tiles per expert
 //   grouped_gemm   for every tile: out[pair] = act(A[pair] . W[expert]^T); A gathered from the step's rows (the way up) or
 //                  read in sorted order (the way down); float32 accumulation on the CUDA cores
-//   routed_combine out[t] = base[t] + sum_s weight[t, s] * y[place of pair (t, s)], float32, in the order of s
+//   routed_combine out[t] = base[t] (times sigmoid of a logit of the row, if one is given) + sum_s weight[t, s] * y[place of
+//                  pair (t, s)], float32, in the order of s
 //
 // The grid of a grouped product is sized for the worst case, ceil(pairs / BM) + experts tiles; blocks beyond the
 // tiles that the plan made return at once.  A pair's result does not depend on where it sits in its tile, so the
@@ -89,6 +92,95 @@ KVB_API int kvb_route_top(const float* logits, int* chosen, float* share, int T,
 KVB_API int kvb_route_top_scores(const float* logits, int* chosen, float* share, int T, int E, int top, int over_all,
                                  cudaStream_t stream) {
     return launch_route_top(logits, chosen, share, T, E, top, over_all ? 1 : 0, stream);
+}
+
+// One warp per row.  Choice scores c = s + correction live in shared memory (one row of experts and one of groups a warp).
+// Groups: `count` runs of E / count neighbours (count 0: none); a group's value is the sum of its two largest c (of its one,
+// if it has one expert); experts outside the `keep` groups with the largest values cannot be chosen.  Ties go to the lower
+// index, of groups and of experts.
+constexpr int ROUTE_WARPS = 4;
+
+// The largest number below `limit` among v[0 .. n), and its lowest place; every lane receives them.
+__device__ __forceinline__ int warp_argmax_below(const float* v, int n, float limit) {
+    const int lane = threadIdx.x & 31;
+    float best = -FLT_MAX;
+    int arg = 0x7fffffff;
+    for (int i = lane; i < n; i += 32)
+        if (v[i] < limit && v[i] > best) { best = v[i]; arg = i; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+        if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+    }
+    return arg;
+}
+
+__global__ void __launch_bounds__(32 * ROUTE_WARPS) route_sigmoid_kernel(const float* __restrict__ logits, int stride,
+                                                                        const float* __restrict__ correction, int* __restrict__ chosen,
+                                                                        float* __restrict__ share, int T, int E, int top, int count,
+                                                                        int keep, float weight_scale) {
+    extern __shared__ float route_s[];          // [ROUTE_WARPS][E + count]
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int r = blockIdx.x * ROUTE_WARPS + warp;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (r >= T) return;
+    float* c = route_s + (size_t)warp * (E + count);
+    float* value = c + E;
+    const float* z = logits + (size_t)r * stride;
+    for (int e = lane; e < E; e += 32) c[e] = 1.f / (1.f + expf(-z[e])) + (correction ? correction[e] : 0.f);
+    __syncwarp();
+    if (count > 0) {
+        const int size = E / count;
+        for (int g = lane; g < count; g += 32) {
+            float a = -FLT_MAX, b = -FLT_MAX;   // the largest and the second
+            for (int i = 0; i < size; ++i) {
+                const float v = c[g * size + i];
+                if (v > a) { b = a; a = v; }
+                else if (v > b) b = v;
+            }
+            value[g] = size > 1 ? a + b : a;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; ++k) {        // a group that stays is marked by an infinite value
+            const int g = warp_argmax_below(value, count, INFINITY);
+            if (lane == 0 && g < count) value[g] = INFINITY;
+            __syncwarp();
+        }
+        for (int e = lane; e < E; e += 32)
+            if (value[e / size] != INFINITY) c[e] = -INFINITY;
+        __syncwarp();
+    }
+    float total = 0.f;
+    for (int s = 0; s < top; ++s) {
+        int e = warp_argmax_below(c, E, INFINITY);
+        if (e >= E) e = 0;                      // nothing comparable is left (scores that are no numbers)
+        if (lane == 0) {
+            c[e] = -INFINITY;
+            chosen[(size_t)r * top + s] = e;
+        }
+        if (lane == (s & 31)) {
+            const float p = 1.f / (1.f + expf(-z[e]));
+            share[(size_t)r * top + s] = p;
+            total += p;
+        }
+        __syncwarp();
+    }
+    total = warp_sum(total) + 1e-20f;
+    for (int s = lane; s < top; s += 32) share[(size_t)r * top + s] *= weight_scale / total;    // the lane that wrote it
+}
+
+// logits [T, stride] float32, the first E columns are the experts'; correction [E] or null; count 0: no groups.
+KVB_API int kvb_route_sigmoid(const float* logits, int stride, const float* correction, int* chosen, float* share, int T, int E, int top,
+                              int count, int keep, float weight_scale, cudaStream_t stream) {
+    if (T <= 0) return KVB_OK;
+    if (E < 1 || E > MOE_MAX_EXPERTS || top < 1 || top > E || stride < E || count < 0) return KVB_ERR_SHAPE;
+    if (count > 0 && (E % count != 0 || keep < 1 || keep > count || top > E / count * keep)) return KVB_ERR_SHAPE;
+    const size_t smem = (size_t)ROUTE_WARPS * (E + count) * sizeof(float);
+    kvb_launch(route_sigmoid_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(32 * ROUTE_WARPS), smem, stream, logits, stride,
+               correction, chosen, share, T, E, top, count, keep, weight_scale);
+    return kvb_launch_status();
 }
 
 // One block.  plan = [tile count | expert offsets (E + 1) | cursors (E)]; tiles[i] = (expert, first sorted row, rows).
@@ -328,29 +420,51 @@ KVB_API int kvb_grouped_gemm_act(int dtype, const void* a, const int* sorted_pai
     return grouped_gemm(dtype, a, sorted_pair, gather_div, w, out, plan, tiles, max_tiles, BM, N, K, act, limit, stream);
 }
 
-// out[t, :] = base[t, :] (if given) + sum_s share[t, s] * y[place[t * top + s], :]
+// out[t, :] = base[t, :] (if given; times sigmoid(gate[t * gate_stride]) if that is) + sum_s share[t, s] * y[place[t * top + s], :]
 template <typename T>
 __global__ void routed_combine_kernel(const T* __restrict__ y, const int* __restrict__ place, const float* __restrict__ share,
-                                      const T* __restrict__ base, T* __restrict__ out, int top, int H) {
+                                      const T* __restrict__ base, const float* __restrict__ gate, int gate_stride, T* __restrict__ out,
+                                      int top, int H) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
+    const float factor = gate ? 1.f / (1.f + expf(-gate[(size_t)t * gate_stride])) : 1.f;
+    if (sizeof(T) == 2 && H % 8 == 0 && (((uintptr_t)y | (uintptr_t)base | (uintptr_t)out) & 15) == 0) {
+        // Eight columns a thread, 16 bytes a load.
+        for (int i = 8 * threadIdx.x; i < H; i += 8 * blockDim.x) {
+            float v[8];
+            const uint4 b4 = base ? *reinterpret_cast<const uint4*>(base + (size_t)t * H + i) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = base ? to_f32<T>(reinterpret_cast<const T*>(&b4)[e]) * factor : 0.f;
+            for (int s = 0; s < top; ++s) {
+                const float p = share[(size_t)t * top + s];
+                const uint4 y4 = *reinterpret_cast<const uint4*>(y + (size_t)place[(size_t)t * top + s] * H + i);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] += p * to_f32<T>(reinterpret_cast<const T*>(&y4)[e]);
+            }
+            uint4 o4;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) reinterpret_cast<T*>(&o4)[e] = from_f32<T>(v[e]);
+            *reinterpret_cast<uint4*>(out + (size_t)t * H + i) = o4;
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        float v = base ? to_f32<T>(base[(size_t)t * H + i]) : 0.f;
+        float v = base ? to_f32<T>(base[(size_t)t * H + i]) * factor : 0.f;
         for (int s = 0; s < top; ++s) v += share[(size_t)t * top + s] * to_f32<T>(y[(size_t)place[(size_t)t * top + s] * H + i]);
         out[(size_t)t * H + i] = from_f32<T>(v);
     }
 }
 
 static int routed_combine(int dtype, const void* y, const int* place, const float* share, const void* base, void* out, int T, int top,
-                          int H, cudaStream_t stream) {
+                          int H, cudaStream_t stream, const float* gate = nullptr, int gate_stride = 0) {
     if (T <= 0) return KVB_OK;
     if (dtype == KVB_F32)
         kvb_launch(routed_combine_kernel<float>, dim3(T), dim3(128), 0, stream, (const float*)y, place, share, (const float*)base,
-                   (float*)out, top, H);
+                   gate, gate_stride, (float*)out, top, H);
     else if (dtype == KVB_BF16)
         kvb_launch(routed_combine_kernel<bf16>, dim3(T), dim3(128), 0, stream, (const bf16*)y, place, share, (const bf16*)base,
-                   (bf16*)out, top, H);
+                   gate, gate_stride, (bf16*)out, top, H);
     else
         return KVB_ERR_DTYPE;
     return kvb_launch_status();
@@ -365,4 +479,11 @@ KVB_API int kvb_routed_combine(int dtype, const void* y, const int* place, const
 KVB_API int kvb_routed_combine_base(int dtype, const void* y, const int* place, const float* share, const void* base, void* out,
                                     int T, int top, int H, cudaStream_t stream) {
     return routed_combine(dtype, y, place, share, base, out, T, top, H, stream);
+}
+
+// The same with `base` multiplied, row by row, by sigmoid(gate[t * gate_stride]) (float32 logits).
+KVB_API int kvb_routed_combine_gated(int dtype, const void* y, const int* place, const float* share, const void* base, const float* gate,
+                                     int gate_stride, void* out, int T, int top, int H, cudaStream_t stream) {
+    if (base == nullptr || gate == nullptr || gate_stride < 1) return KVB_ERR_SHAPE;
+    return routed_combine(dtype, y, place, share, base, out, T, top, H, stream, gate, gate_stride);
 }

@@ -327,7 +327,7 @@ KVB_API int kvb_qkv_rope_append(int dtype, const void* qkv, const float* bias, c
 // Dk wide with zeros after their D numbers (keys as wide as values, so that kernels for equal sizes serve them; the
 // zeros add nothing to a score).  `Dvs` >= Dv: values are stored Dvs wide with zeros after their Dv numbers.  `qt_every` > 0:
 // the queries of a row at position p are multiplied by 1 + qt_coef * ln(floor((p + 1) / qt_every) + 1) (float32), after
-// norm and rotation.
+// norm and rotation.  Hkv 0 (without write_kv): rows of queries alone, for a layer that reads another layer's keys.
 enum { QKV_NORM = 1, QKV_NORM_ALL = 2, QKV_NORM_AFTER = 4 };
 enum { QKV_MIX_NONE = 0, QKV_MIX_SOURCE = 1, QKV_MIX_BLEND = 2 };
 
@@ -378,7 +378,7 @@ __global__ void qkv_norm_rope_append_kernel(const T* __restrict__ qkv, int row_s
             sk += v * v;
         }
         inv_q = 1.f / sqrtf(block_sum(sq, scratch) / (float)(Hq * D) + eps);
-        inv_k = 1.f / sqrtf(block_sum(sk, scratch) / (float)(Hkv * D) + eps);
+        if (Hkv > 0) inv_k = 1.f / sqrtf(block_sum(sk, scratch) / (float)(Hkv * D) + eps);
     }
     float* mine = head_s + (size_t)warp * 2 * D;
     float* turned = mine + D;
@@ -443,6 +443,198 @@ __global__ void qkv_norm_rope_append_kernel(const T* __restrict__ qkv, int row_s
     }
 }
 
+// The same for bfloat16 rows whose norm runs over the whole query (key) projection with weights, in steps of eight numbers:
+// a block takes ROWS consecutive rows.  A thread reads 16 bytes at a time, adds the biases, leaves (x + b) * w in shared
+// memory and its squares in two sums a row (queries, keys); after one barrier for the sums every thread takes chunks again,
+// rotates them with their partner chunks from shared memory and multiplies by the row's inverse root mean square on the way
+// out (the rotation is linear, so the order does not matter).  Values pass straight through.  What does not depend on the
+// product before this kernel - positions, pages, angles, the first chunk's biases and weights - is fetched before the wait.
+// A row's additions are the same whatever ROWS: the number of threads follows from the row's width alone.
+template <int ROWS>
+__global__ void __launch_bounds__(ROWS == 1 ? 1024 : 512)
+qkv_whole_norm_rope_append_kernel(const bf16* __restrict__ qkv, int row_stride, const float* __restrict__ bias,
+                                                  const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                                                  const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_half,
+                                                  int table_len, const int* __restrict__ positions, const int* __restrict__ row_segment,
+                                                  const int* __restrict__ block_table, int table_stride, bf16* __restrict__ k_pages,
+                                                  bf16* __restrict__ v_pages, bf16* __restrict__ q_out, int T, int Hq, int Hkv, int D,
+                                                  int Dv, int Dk, int Dvs, int page_size, int write_kv, int* __restrict__ err) {
+    extern __shared__ __align__(16) float row_s[];      // [ROWS][qk]: (x + b) * w, then [ROWS][2 rot_half]: cos, sin
+    __shared__ float part_s[32][2 * ROWS];              // each warp's sums of squares
+    __shared__ float inv_s[2 * ROWS];
+    __shared__ long long page_row_s[ROWS];              // (page, slot) of the row's keys and values, counted in tokens; -1: none
+    if (ROWS == 1) pdl_launch_dependents();             // a few small blocks: the successor may come onto the SMs at once
+    const int r0 = blockIdx.x * ROWS;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+    const int q_width = Hq * D, qk = (Hq + Hkv) * D, rot = 2 * rot_half;
+    const int qk_chunks = qk >> 3, chunks = qk_chunks + (write_kv ? Hkv * Dv >> 3 : 0);
+    float* angles = row_s + ROWS * qk;
+    if (tid < ROWS) {
+        const int r = r0 + tid;
+        long long at = -1;
+        if (r < T && write_kv) {
+            const int pos = positions[r];
+            const int page = block_table[(size_t)row_segment[r] * table_stride + pos / page_size];
+            if (page < 0) atomicOr(err, KVB_DEV_BAD_PAGE);
+            else at = (long long)page * Hkv * page_size + pos % page_size;
+        }
+        page_row_s[tid] = at;
+    }
+    for (int i = tid; i < ROWS * rot; i += blockDim.x) {
+        const int row = i / rot, j = i - row * rot, r = r0 + row;
+        float v = 0.f;
+        if (r < T) {
+            const int pos = positions[r];
+            const bool pos_ok = pos >= 0 && pos < table_len;
+            if (!pos_ok && j == 0) atomicOr(err, KVB_DEV_BAD_POS);
+            const int p = pos_ok ? pos : 0;
+            v = j < rot_half ? cos_t[(size_t)p * rot_half + j] : sin_t[(size_t)p * rot_half + j - rot_half];
+        }
+        angles[i] = v;
+    }
+    float b[8], w[8];
+    auto constants = [&](int c) {                        // biases and weights of chunk c
+        const int at = 8 * c;
+        const float* ws = at < q_width ? q_w + at : k_w + at - q_width;
+#pragma unroll
+        for (int e = 0; e < 8; e += 4) {
+            const float4 b4 = bias ? *reinterpret_cast<const float4*>(bias + at + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+            b[e] = b4.x; b[e + 1] = b4.y; b[e + 2] = b4.z; b[e + 3] = b4.w;
+            const float4 w4 = c < qk_chunks ? *reinterpret_cast<const float4*>(ws + e) : make_float4(1.f, 1.f, 1.f, 1.f);
+            w[e] = w4.x; w[e + 1] = w4.y; w[e + 2] = w4.z; w[e + 3] = w4.w;
+        }
+    };
+    if (tid < chunks) constants(tid);
+    pdl_wait();
+    if (ROWS != 1) pdl_launch_dependents();
+    __syncthreads();                                     // the rows' pages
+    float sums[2 * ROWS];
+#pragma unroll
+    for (int i = 0; i < 2 * ROWS; ++i) sums[i] = 0.f;
+    for (int c = tid; c < chunks; c += blockDim.x) {
+        if (c != tid) constants(c);
+        uint4 raw[ROWS];
+#pragma unroll
+        for (int row = 0; row < ROWS; ++row)
+            raw[row] = *reinterpret_cast<const uint4*>(qkv + (size_t)min(r0 + row, T - 1) * row_stride + 8 * c);
+#pragma unroll
+        for (int row = 0; row < ROWS; ++row) {
+            const uint32_t in[4] = {raw[row].x, raw[row].y, raw[row].z, raw[row].w};
+            float x[8];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&in[k]));
+                x[2 * k] = f.x + b[2 * k];
+                x[2 * k + 1] = f.y + b[2 * k + 1];
+            }
+            if (c < qk_chunks) {
+                float ss = 0.f;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+                if (8 * c < q_width) sums[2 * row] += ss; else sums[2 * row + 1] += ss;
+                float4* dst = reinterpret_cast<float4*>(row_s + row * qk + 8 * c);
+                dst[0] = make_float4(x[0] * w[0], x[1] * w[1], x[2] * w[2], x[3] * w[3]);
+                dst[1] = make_float4(x[4] * w[4], x[5] * w[5], x[6] * w[6], x[7] * w[7]);
+            } else if (page_row_s[row] >= 0) {
+                const int at = 8 * (c - qk_chunks), hk = at / Dv, d = at - hk * Dv;
+                uint32_t o[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const __nv_bfloat162 v = __floats2bfloat162_rn(x[2 * k], x[2 * k + 1]);
+                    o[k] = *reinterpret_cast<const uint32_t*>(&v);
+                }
+                *reinterpret_cast<uint4*>(v_pages + ((size_t)page_row_s[row] + (size_t)hk * page_size) * Dvs + d) = make_uint4(o[0], o[1], o[2], o[3]);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2 * ROWS; ++i) {
+        const float s = warp_sum(sums[i]);
+        if (lane == 0) part_s[warp][i] = s;
+    }
+    __syncthreads();
+    if (tid < 2 * ROWS) {
+        float total = 0.f;
+        for (int k = 0; k < warps; ++k) total += part_s[k][tid];
+        const int n = (tid & 1) ? Hkv * D : q_width;
+        inv_s[tid] = n > 0 ? 1.f / sqrtf(total / (float)n + eps) : 0.f;
+    }
+    __syncthreads();
+    const int per_head = Dk >> 3;                        // chunks of a stored head: its own, then zeros
+    for (int c = tid; c < (Hq + (write_kv ? Hkv : 0)) * per_head; c += blockDim.x) {
+        const int head = c / per_head, d = 8 * (c - head * per_head);
+        const bool is_q = head < Hq;
+#pragma unroll
+        for (int row = 0; row < ROWS; ++row) {
+            if (r0 + row >= T || (!is_q && page_row_s[row] < 0)) continue;
+            float x[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = 0.f;
+            if (d < D) {
+                const float* own = row_s + row * qk + head * D + d;
+#pragma unroll
+                for (int e = 0; e < 8; e += 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(own + e);
+                    x[e] = v.x; x[e + 1] = v.y; x[e + 2] = v.z; x[e + 3] = v.w;
+                }
+                if (d < rot) {
+                    const bool low = d < rot_half;
+                    const float* partner = low ? own + rot_half : own - rot_half;
+                    const float* cs = angles + row * rot + (low ? d : d - rot_half);
+                    const float* sn = cs + rot_half;
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) x[e] = low ? x[e] * cs[e] - partner[e] * sn[e] : x[e] * cs[e] + partner[e] * sn[e];
+                }
+                const float inv = inv_s[2 * row + (is_q ? 0 : 1)];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[e] *= inv;
+            }
+            uint32_t o[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const __nv_bfloat162 v = __floats2bfloat162_rn(x[2 * k], x[2 * k + 1]);
+                o[k] = *reinterpret_cast<const uint32_t*>(&v);
+            }
+            bf16* dst = is_q ? q_out + ((size_t)(r0 + row) * Hq + head) * Dk
+                             : k_pages + ((size_t)page_row_s[row] + (size_t)(head - Hq) * page_size) * Dk;
+            *reinterpret_cast<uint4*>(dst + d) = make_uint4(o[0], o[1], o[2], o[3]);
+        }
+    }
+    if (write_kv && Dvs > Dv) {
+        const int pad = (Dvs - Dv) >> 3;
+        for (int i = tid; i < ROWS * Hkv * pad; i += blockDim.x) {
+            const int row = i / (Hkv * pad), at = i - row * Hkv * pad, hk = at / pad, d = Dv + 8 * (at - hk * pad);
+            if (page_row_s[row] >= 0)
+                *reinterpret_cast<uint4*>(v_pages + ((size_t)page_row_s[row] + (size_t)hk * page_size) * Dvs + d) = make_uint4(0u, 0u, 0u, 0u);
+        }
+    }
+}
+
+// KVB_ERR_LIMIT: sizes or addresses this kernel does not take (the caller has another).
+static int launch_whole_norm(const bf16* qkv, int row_stride, const float* bias, const float* q_w, const float* k_w, float eps,
+                             const float* cos_t, const float* sin_t, int rot_half, int table_len, const int* positions,
+                             const int* row_segment, const int* block_table, int table_stride, bf16* k_pages, bf16* v_pages, bf16* q_out,
+                             int T, int Hq, int Hkv, int D, int Dv, int Dk, int Dvs, int page_size, int write_kv, int* err,
+                             cudaStream_t stream) {
+    const uintptr_t addresses = (uintptr_t)qkv | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)q_out | (uintptr_t)bias | (uintptr_t)q_w | (uintptr_t)k_w;
+    if ((addresses & 15) || ((row_stride | D | Dv | Dk | Dvs | rot_half) & 7)) return KVB_ERR_LIMIT;
+    const int qk = (Hq + Hkv) * D;
+    const int chunks = (qk + (write_kv ? Hkv * Dv : 0)) / 8;
+    const int threads = chunks >= 1024 ? 1024 : (chunks + 31) / 32 * 32;
+    constexpr int ROWS = 4;
+    const size_t one = (size_t)(qk + 2 * rot_half) * sizeof(float);
+    if (one > 46 * 1024) return KVB_ERR_LIMIT;           // 48 KB without an attribute, some of it the kernel's own
+    if (T >= 256 && ROWS * one <= 46 * 1024 && threads <= 512)
+        kvb_launch(qkv_whole_norm_rope_append_kernel<ROWS>, dim3((T + ROWS - 1) / ROWS), dim3(threads), ROWS * one, stream, qkv, row_stride,
+                   bias, q_w, k_w, eps, cos_t, sin_t, rot_half, table_len, positions, row_segment, block_table, table_stride, k_pages,
+                   v_pages, q_out, T, Hq, Hkv, D, Dv, Dk, Dvs, page_size, write_kv, err);
+    else
+        kvb_launch(qkv_whole_norm_rope_append_kernel<1>, dim3(T), dim3(threads), one, stream, qkv, row_stride, bias, q_w, k_w, eps, cos_t,
+                   sin_t, rot_half, table_len, positions, row_segment, block_table, table_stride, k_pages, v_pages, q_out, T, Hq, Hkv, D,
+                   Dv, Dk, Dvs, page_size, write_kv, err);
+    return kvb_launch_status();
+}
+
 // `norm_flags`: QKV_NORM - queries and keys are normalised (weights q_w / k_w, or none); QKV_NORM_ALL - over a row's whole
 // query (key) projection, all heads at once, with weights of that size, instead of per head with weights of D numbers
 // that the heads share; QKV_NORM_AFTER - after the rotation instead of before it (per head only).  `mix_mode`:
@@ -455,11 +647,17 @@ KVB_API int kvb_qkv_norm_rope_append(int dtype, const void* qkv, int row_stride,
                                      const float* lam, int Dvs, float qt_coef, int qt_every, int* err, cudaStream_t stream) {
     if (T <= 0) return KVB_OK;
     if (2 * rot_half > D || rot_half < 0 || Dv < 1 || Dk < D || Dvs < Dv || qt_every < 0 || row_stride < (Hq + Hkv) * D + Hkv * Dv ||
-        (q_w == nullptr) != (k_w == nullptr))
+        Hq < 1 || Hkv < 0 || (Hkv == 0 && (write_kv || mix_mode != 0)) || (Hkv > 0 && (q_w == nullptr) != (k_w == nullptr)))
         return KVB_ERR_SHAPE;
     if ((norm_flags & QKV_NORM_ALL) && (norm_flags & QKV_NORM_AFTER)) return KVB_ERR_SHAPE;
     if (mix_mode < 0 || mix_mode > QKV_MIX_BLEND || (mix_mode != 0 && kept == nullptr) || (mix_mode == QKV_MIX_BLEND && lam == nullptr))
         return KVB_ERR_SHAPE;
+    if (dtype == KVB_BF16 && norm_flags == (QKV_NORM | QKV_NORM_ALL) && mix_mode == 0 && qt_every == 0 && q_w != nullptr) {
+        const int rc = launch_whole_norm((const bf16*)qkv, row_stride, bias, q_w, k_w, eps, cos_t, sin_t, rot_half, table_len, positions,
+                                         row_segment, block_table, table_stride, (bf16*)k_pages, (bf16*)v_pages, (bf16*)q_out, T, Hq, Hkv,
+                                         D, Dv, Dk, Dvs, page_size, write_kv, err, stream);
+        if (rc != KVB_ERR_LIMIT) return rc;
+    }
     const int warps = Hq + Hkv >= 8 ? 8 : 4;
     const size_t smem = ((size_t)warps * 2 * D + 33) * sizeof(float);
     if (smem > 48 * 1024) return KVB_ERR_LIMIT;

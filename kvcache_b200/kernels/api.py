@@ -17,7 +17,7 @@ import torch
 
 from ..parts.base import PagedKVView, StepBatch
 from . import build
-from .attention_plan import PagedAttentionPlanner
+from .attention_plan import PREFILL_MIN_KEY_TILES, TC_MIN_KEY_TILES, PagedAttentionPlanner
 from .latent_plan import LatentAttentionPlanner
 
 _c_int, _c_float, _c_void_p, _c_longlong = ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_longlong
@@ -43,7 +43,7 @@ class KernelSet:
     qkv_rope_append(qkv[T,(Hq+2Hkv)D], bias, cos, sin, batch, kv, q_out[T,Hq*D]):
         adds the bias, rotates queries and keys by the row's position, writes the queries to
         q_out and, if kv.writes, keys and values into their cache pages
-    paged_attention(q[T,Hq*D], batch, kv, out[T,Hq*D], scale): causal (windowed if kv.spec.window)
+    paged_attention(q[T,Hq*D], batch, kv, out[T,Hq*D], scale): causal (within a window or chunk if kv.spec has one)
         softmax(scale * q.k) v over the keys of the row's request, from the pages
     rope_append_attention(qkv, bias, cos, sin, batch, kv, out, num_heads, scale, workspace) -> bool   (optional)
         both of the above in one launch where the set has a kernel for the step at hand; False: nothing was
@@ -92,7 +92,8 @@ _SIGNATURES = {
         "kvb_token_shift": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                             _c_int, _c_int, _c_void_p],
         "kvb_activation": [_c_int, _c_void_p, _c_longlong, _c_int, _c_float, _c_void_p],
-        "kvb_add_rmsnorm": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
+        "kvb_add_norm": [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float,
+                         _c_void_p],
         "kvb_silu_mul": [_c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_gated_act": [_c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
     },
@@ -164,6 +165,9 @@ _SIGNATURES = {
         "kvb_grouped_gemm_act": [_c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                  _c_int, _c_int, _c_int, _c_float, _c_void_p],
         "kvb_routed_combine_base": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
+        "kvb_route_sigmoid": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+        "kvb_routed_combine_gated": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int,
+                                     _c_void_p],
         "kvb_routed_plan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
         "kvb_grouped_gemm": [_c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                              _c_int, _c_int, _c_int, _c_void_p],
@@ -186,7 +190,7 @@ _SIGNATURES = {
         "kvb_gemm_wstream_gated": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     },
     "gemm_tcgen05": {
-        "kvb_gemm_tcgen05": [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+        "kvb_gemm_tcgen05": [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     },
     "attention_flash": {
         "kvb_flash_head_dim": [],
@@ -203,13 +207,13 @@ _SIGNATURES = {
                                  _c_void_p, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p],
         "kvb_flash_prefill": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p,
                               _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p,
-                              _c_int, _c_void_p, _c_float, _c_void_p],
+                              _c_int, _c_void_p, _c_float, _c_int, _c_void_p],
     },
     "attention_tc": {
         "kvb_attention_tc_head_dim": [],
         "kvb_attention_tc": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p,
                              _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                             _c_void_p, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p],
+                             _c_void_p, _c_int, _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p],
     },
     "primitive_costs": {
         "kvb_primitive_costs_count": [],
@@ -296,6 +300,9 @@ class CudaKernels(KernelSet):
         # 0.5B shape: the mma.sync kernel is ahead at 128 and 256 rows (1.09 / 1.24 ms a step against 1.14 / 1.28),
         # the tensor-memory kernel from 512 rows on (1.56 against 1.69 ms).
         self.tc_attention_min_rows: Optional[int] = 384
+        # A window or chunks may leave a tile of a portion fewer key tiles than its units were planned for: a unit keeps at
+        # least this many (what kernels/attention_plan.py plans with).
+        self.tc_unit_min_tiles, self.prefill_unit_min_tiles = TC_MIN_KEY_TILES, PREFILL_MIN_KEY_TILES
         self.flash_attention = True          # bfloat16, head sizes 16..128: tensor-core kernels
         # Decode steps of at least this many requests: bias, rotation and append inside the TMA decode kernel (None: never).
         # Measured on 24 layers of the 0.5B shape at 4,096 tokens of context, a step with the kernel against a step with
@@ -528,14 +535,19 @@ class CudaKernels(KernelSet):
         return (torch.arange(num_heads_total)[:, None] * head_dim + within[None, :]).reshape(-1)
 
     def add_rmsnorm(self, h: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
-                    out: torch.Tensor, rows: Optional[torch.Tensor] = None, delta_scale: Optional[torch.Tensor] = None) -> None:
-        """`delta_scale` (float32 [H]): delta is multiplied by it, channel by channel, before the add."""
+                    out: torch.Tensor, rows: Optional[torch.Tensor] = None, delta_scale: Optional[torch.Tensor] = None,
+                    delta_bias: Optional[torch.Tensor] = None, centred: bool = False) -> None:
+        """h += (delta + `delta_bias`) * `delta_scale` (float32 [H] each, either may be None), then the norm; `centred`: the mean of
+        a row is taken off first and the squares are those of the deviations."""
         n_out, H = out.shape
-        if delta_scale is not None and (delta_scale.dtype != torch.float32 or delta_scale.numel() != H):
-            raise KernelError("add_rmsnorm: the delta's scale is one float32 number per channel")
+        for v in (delta_scale, delta_bias):
+            if v is not None and (v.dtype != torch.float32 or v.numel() != H):
+                raise KernelError("add_rmsnorm: the delta's scale and bias are one float32 number per channel")
+        if delta is None:
+            delta_scale = delta_bias = None
         self._count("add_rmsnorm")
-        _check(self._elementwise.kvb_add_rmsnorm(_dtype_code(out.dtype), _ptr(h), _ptr(delta), _ptr(delta_scale if delta is not None else None),
-                                                 _ptr(weight), _ptr(out), _ptr(rows), n_out, H, float(eps), self._stream()),
+        _check(self._elementwise.kvb_add_norm(_dtype_code(out.dtype), 1 if centred else 0, _ptr(h), _ptr(delta), _ptr(delta_scale),
+                                              _ptr(delta_bias), _ptr(weight), _ptr(out), _ptr(rows), n_out, H, float(eps), self._stream()),
                "add_rmsnorm")
 
     GATED_ACTIVATIONS = {"silu": 0, "clamped_swiglu": 1}
@@ -558,8 +570,9 @@ class CudaKernels(KernelSet):
     def gate_up_act(self, x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, workspace, interleaved: bool,
                     activation: str = "silu", limit: float = 0.0) -> None:
         """out[M, I] = act(x Wg^T, x Wu^T) (see `silu_mul`); `w_gate_up` [2 I, K] holds gate and up rows one after the
-        other, or interleaved in eights (see csrc/gemm_skinny.cu).  The clamped activation is in the epilogue of the two
-        weight-streaming products (steps of few rows); with more rows it takes the product and the activation kernel."""
+        other, or interleaved in eights (see csrc/gemm_skinny.cu).  Either activation is in the epilogue of the two
+        weight-streaming products (steps of few rows) and of the tensor-memory product where its tiles fill the GPU; in
+        between it takes the library product and the activation kernel."""
         M, K = x.shape
         I = out.shape[1]
         if activation != "silu":
@@ -575,6 +588,12 @@ class CudaKernels(KernelSet):
                 _check(self._gemm_ws.kvb_gemm_wstream_gated(_dtype_code(out.dtype), _ptr(x), _ptr(w_gate_up), _ptr(out), M, 2 * I, K,
                                                             float(limit), _ptr(self.error_word), self._stream()),
                        "gate_up_act (wstream, clamped)")
+                return
+            if interleaved and self._tcgen05(x, w_gate_up, out, fused=True):
+                self._count("gemm_tcgen05")
+                _check(self._gemm_tc.kvb_gemm_tcgen05(_dtype_code(out.dtype), 1, _ptr(x), _ptr(w_gate_up), _ptr(None), _ptr(out), M,
+                                                      2 * I, K, float(limit), _ptr(self.error_word), self._stream()),
+                       "gate_up_act (tcgen05, clamped)")
                 return
             gate_up = workspace.buffer("ffn.gate_up", (M, 2 * I), out.dtype)
             self.linear(x, w_gate_up, gate_up)
@@ -593,7 +612,7 @@ class CudaKernels(KernelSet):
         if interleaved and self._tcgen05(x, w_gate_up, out, fused=True):
             self._count("gemm_tcgen05")
             _check(self._gemm_tc.kvb_gemm_tcgen05(_dtype_code(out.dtype), 1, _ptr(x), _ptr(w_gate_up), _ptr(None), _ptr(out), M,
-                                                  2 * I, K, _ptr(self.error_word), self._stream()), "gate_up_act (tcgen05)")
+                                                  2 * I, K, 0.0, _ptr(self.error_word), self._stream()), "gate_up_act (tcgen05)")
             return
         gate_up = workspace.buffer("ffn.gate_up", (M, 2 * I), out.dtype)
         self.linear(x, w_gate_up, gate_up)
@@ -648,7 +667,7 @@ class CudaKernels(KernelSet):
         if self._tcgen05(x, w, out):
             self._count("gemm_tcgen05")
             _check(self._gemm_tc.kvb_gemm_tcgen05(_dtype_code(out.dtype), 0, _ptr(x), _ptr(w), _ptr(bias), _ptr(out), M, N, K,
-                                                  _ptr(self.error_word), self._stream()), "linear (tcgen05)")
+                                                  0.0, _ptr(self.error_word), self._stream()), "linear (tcgen05)")
             return
         if x.dtype == torch.bfloat16 and self.bf16_gemm != "simt":
             # Library matrix product, as the reference's cublasGemmEx (apps/qwen_serve.cu:27-39).
@@ -668,7 +687,8 @@ class CudaKernels(KernelSet):
                         sin: Optional[torch.Tensor], batch: StepBatch, kv: PagedKVView, q_out: torch.Tensor,
                         num_heads: int, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
                         norm_eps: float = 0.0, key_dim: Optional[int] = None, norm_scope: str = "head",
-                        norm_after_rotation: bool = False, value_mix=None, q_temperature=None, value_dim: Optional[int] = None) -> None:
+                        norm_after_rotation: bool = False, value_mix=None, q_temperature=None, value_dim: Optional[int] = None,
+                        queries_only: bool = False) -> None:
         """`q_norm` / `k_norm` (float32 [key_dim]): queries and keys are divided by their root mean square per head and
         multiplied by these before the rotation.  `norm_eps` > 0 without weights: the division alone.  `norm_scope` "all":
         the root mean square runs over a row's whole query (key) projection and the weights have that size.
@@ -677,7 +697,8 @@ class CudaKernels(KernelSet):
         of `qkv` may carry further columns after [q | k | v].  `key_dim` < `kv.spec.head_dim`: queries and keys have
         `key_dim` numbers in `qkv` and are stored `kv.spec.head_dim` wide, with zeros after them.  `value_dim` <
         `kv.spec.v_head_dim`: likewise for the values.  `q_temperature` = (coef, every): the queries of a row at position p are
-        multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+        multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  `queries_only`: rows of queries alone, nothing is appended (a
+        layer that reads the cache entry of another)."""
         T = qkv.shape[0]
         spec = kv.spec
         rot_half = 0 if cos is None else cos.shape[1]
@@ -686,7 +707,10 @@ class CudaKernels(KernelSet):
         normed = q_norm is not None or norm_eps > 0.0
         Dv = spec.v_head_dim if value_dim is None else int(value_dim)
         qt_coef, qt_every = q_temperature if q_temperature is not None else (0.0, 0)
-        if (normed or value_mix is not None or spec.v_head_dim != spec.head_dim or D != spec.head_dim or Dv != spec.v_head_dim
+        if queries_only and kv.writes:
+            raise KernelError("qkv_rope_append: rows of queries alone, but the call writes the cache")
+        Hkv = 0 if queries_only else spec.num_kv_heads
+        if (normed or queries_only or value_mix is not None or spec.v_head_dim != spec.head_dim or D != spec.head_dim or Dv != spec.v_head_dim
                 or q_temperature is not None or qkv.shape[1] != (num_heads + 2 * spec.num_kv_heads) * spec.head_dim):
             flags = (1 if normed else 0) | (2 if normed and norm_scope == "all" else 0) | (4 if normed and norm_after_rotation else 0)
             kept, lam = value_mix if value_mix is not None else (None, None)
@@ -697,7 +721,7 @@ class CudaKernels(KernelSet):
             _check(self._rope.kvb_qkv_norm_rope_append(
                 _dtype_code(qkv.dtype), _ptr(qkv), qkv.shape[1], _ptr(bias), _ptr(q_norm), _ptr(k_norm), float(norm_eps), flags,
                 _ptr(cos), _ptr(sin), rot_half, table_len, _ptr(batch.positions), _ptr(batch.row_segment), _ptr(kv.block_table),
-                kv.block_table.shape[1], _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(q_out), T, num_heads, spec.num_kv_heads,
+                kv.block_table.shape[1], _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(q_out), T, num_heads, Hkv,
                 D, Dv, spec.head_dim, kv.page_size, 1 if kv.writes else 0, mix_mode, _ptr(kept), _ptr(lam), spec.v_head_dim,
                 float(qt_coef), int(qt_every), _ptr(self.error_word), self._stream()), "qkv_norm_rope_append")
             return
@@ -760,23 +784,25 @@ class CudaKernels(KernelSet):
         _check(lib.kvb_flash_decode_tma(
             None, _ptr(out), _ptr(kv.k_pages), _ptr(kv.v_pages), kv.k_pages.shape[0], _ptr(kv.block_table),
             kv.block_table.shape[1], None, n, _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_kv_len),
-            num_heads, Hkv, kv.page_size, spec.window or 0, nsplit, float(scale), _ptr(qkv), _ptr(bias), _ptr(cos), _ptr(sin),
+            num_heads, Hkv, kv.page_size, spec.reach, nsplit, float(scale), _ptr(qkv), _ptr(bias), _ptr(cos), _ptr(sin),
             0 if cos is None else cos.shape[1], 0 if cos is None else cos.shape[0], 1, None, None, None, 0, None, 0.0, _ptr(self.error_word),
             self._stream()), "flash_decode_tma (rotation and append fused)")
         return True
 
     def paged_attention(self, q: torch.Tensor, batch: StepBatch, kv: PagedKVView, out: torch.Tensor,
                         num_heads: int, scale: float, workspace=None, sink: Optional[torch.Tensor] = None,
-                        score_cap: Optional[float] = None, slopes: Optional[torch.Tensor] = None) -> None:
+                        score_cap: Optional[float] = None, slopes: Optional[torch.Tensor] = None, reach: Optional[int] = None) -> None:
         """`sink` (float32 [num_heads]): the softmax's denominator also holds exp(sink[h]), a key without a value.
         `kv.spec.keep_first` (with a window): the request's first keys stay visible to every later query.
         `score_cap`: a score (after the scale) becomes cap tanh(score / cap).  `slopes` (float32 [num_heads]): a key i - j
-        tokens back then loses slopes[h] (i - j)."""
+        tokens back then loses slopes[h] (i - j).  `reach` (see parts.base.reach_code; None: the cache entry's own): which keys a
+        query sees, for a layer that reads a cache entry that keeps more than the layer sees."""
         T = q.shape[0]
         spec = kv.spec
+        reach = spec.reach if reach is None else int(reach)
         D, Hkv = spec.head_dim, spec.num_kv_heads
         plan = batch.plans.get(PagedAttentionPlanner.name)
-        keep = spec.keep_first if spec.window else 0
+        keep = spec.keep_first if reach > 0 else 0
         fast = (self.flash_attention and q.dtype == torch.bfloat16 and spec.v_head_dim == D and D % 16 == 0 and D <= 128
                 and num_heads // Hkv <= 16 and workspace is not None and plan is not None)
         # Capped or biased scores: the tensor-core kernels (all but the cluster decode kernel without TMA) make the whole score
@@ -792,7 +818,7 @@ class CudaKernels(KernelSet):
             _check(self._attn_generic.kvb_paged_attention_ext(
                 _dtype_code(q.dtype), _ptr(q), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table), kv.block_table.shape[1],
                 _ptr(batch.positions), _ptr(batch.row_segment), _ptr(out), T, num_heads, Hkv, D, spec.v_head_dim, kv.page_size,
-                spec.window or 0, keep, _ptr(sink), float(scale), cap, _ptr(slopes), _ptr(self.error_word), self._stream()),
+                reach, keep, _ptr(sink), float(scale), cap, _ptr(slopes), _ptr(self.error_word), self._stream()),
                 "paged_attention")
             return
         # The cluster decode kernel knows neither a sink nor kept first keys nor biased scores: with them, and where the TMA
@@ -803,7 +829,7 @@ class CudaKernels(KernelSet):
             _check(self._attn_generic.kvb_paged_attention_sink(
                 _dtype_code(q.dtype), _ptr(q), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table), kv.block_table.shape[1],
                 _ptr(batch.positions), _ptr(batch.row_segment), _ptr(out), T, num_heads, Hkv, D, spec.v_head_dim, kv.page_size,
-                spec.window or 0, spec.keep_first if spec.window else 0, _ptr(sink), float(scale), _ptr(self.error_word),
+                reach, keep, _ptr(sink), float(scale), _ptr(self.error_word),
                 self._stream()), "paged_attention")
             return
         if spec.v_head_dim != D:
@@ -812,7 +838,7 @@ class CudaKernels(KernelSet):
             _check(self._attn_generic.kvb_paged_attention_kv(
                 _dtype_code(q.dtype), _ptr(q), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table), kv.block_table.shape[1],
                 _ptr(batch.positions), _ptr(batch.row_segment), _ptr(out), T, num_heads, Hkv, D, spec.v_head_dim, kv.page_size,
-                spec.window or 0, float(scale), _ptr(self.error_word), self._stream()), "paged_attention")
+                reach, float(scale), _ptr(self.error_word), self._stream()), "paged_attention")
             return
         if fast:
             lib = self._flash_library(D)
@@ -831,7 +857,8 @@ class CudaKernels(KernelSet):
                     _ptr(q), _ptr(out), _ptr(kv.k_pages), _ptr(kv.v_pages), kv.k_pages.shape[0], _ptr(kv.block_table),
                     kv.block_table.shape[1], _ptr(lists["tc_units"]), units, _ptr(scratch), _ptr(tickets),
                     _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_kv_len), T, num_heads, Hkv, kv.page_size,
-                    spec.window or 0, float(scale), _ptr(sink), keep, _ptr(slopes), cap, _ptr(self.error_word), self._stream()),
+                    reach, float(scale), _ptr(sink), keep, _ptr(slopes), cap, self.tc_unit_min_tiles, _ptr(self.error_word),
+                    self._stream()),
                     "attention_tc")
             elif counts["prefill_units"]:
                 units = counts["prefill_units"]
@@ -841,8 +868,8 @@ class CudaKernels(KernelSet):
                 _check(lib.kvb_flash_prefill(
                     _ptr(q), _ptr(out), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table), kv.block_table.shape[1],
                     _ptr(lists["prefill_units"]), units, _ptr(batch.seg_q_start), _ptr(batch.seg_q_len),
-                    _ptr(batch.seg_kv_len), _ptr(scratch), _ptr(tickets), num_heads, Hkv, kv.page_size, spec.window or 0,
-                    float(scale), _ptr(sink), keep, _ptr(slopes), cap, self._stream()), "flash_prefill")
+                    _ptr(batch.seg_kv_len), _ptr(scratch), _ptr(tickets), num_heads, Hkv, kv.page_size, reach,
+                    float(scale), _ptr(sink), keep, _ptr(slopes), cap, self.prefill_unit_min_tiles, self._stream()), "flash_prefill")
             n = counts["decode_items"]
             items = lists["decode_items"]
             if n:
@@ -875,7 +902,7 @@ class CudaKernels(KernelSet):
                             _ptr(kv.block_table), kv.block_table.shape[1],
                             _ptr(None if n == batch.num_segments else items), n,   # every segment, in order: no list
                             _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_kv_len), num_heads, Hkv,
-                            kv.page_size, spec.window or 0, nsplit, float(scale), None, None, None, None, 0, 0,
+                            kv.page_size, reach, nsplit, float(scale), None, None, None, None, 0, 0,
                             nsuper, _ptr(scratch), _ptr(tickets), _ptr(sink), keep, _ptr(slopes), cap, _ptr(self.error_word),
                             self._stream()), "flash_decode_tma")
                         return
@@ -883,7 +910,7 @@ class CudaKernels(KernelSet):
                     _check(lib.kvb_flash_decode_cluster(
                         _ptr(q), _ptr(out), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table),
                         kv.block_table.shape[1], _ptr(items), n, _ptr(batch.seg_q_start),
-                        _ptr(batch.seg_q_len), _ptr(batch.seg_kv_len), num_heads, Hkv, kv.page_size, spec.window or 0,
+                        _ptr(batch.seg_q_len), _ptr(batch.seg_kv_len), num_heads, Hkv, kv.page_size, reach,
                         nsplit, float(scale), self._stream()), "flash_decode_cluster")
                     return
                 nsplit = max(1, min(32, 2 * self.decode_ctas_wanted // (n * Hkv), tiles // self.decode_min_tiles))
@@ -893,14 +920,14 @@ class CudaKernels(KernelSet):
                 _check(lib.kvb_flash_decode(
                     _ptr(q), _ptr(out), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table), kv.block_table.shape[1],
                     _ptr(items), n, _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_kv_len),
-                    _ptr(scratch), _ptr(tickets), num_heads, Hkv, kv.page_size, spec.window or 0, nsplit, float(scale),
+                    _ptr(scratch), _ptr(tickets), num_heads, Hkv, kv.page_size, reach, nsplit, float(scale),
                     _ptr(sink), keep, _ptr(slopes), cap, self._stream()), "flash_decode")
             return
         self._count("attention_generic")
         _check(self._attn_generic.kvb_paged_attention_generic(
             _dtype_code(q.dtype), _ptr(q), _ptr(kv.k_pages), _ptr(kv.v_pages), _ptr(kv.block_table),
             kv.block_table.shape[1], _ptr(batch.positions), _ptr(batch.row_segment), _ptr(out), T, num_heads,
-            spec.num_kv_heads, spec.head_dim, kv.page_size, spec.window or 0, float(scale),
+            spec.num_kv_heads, spec.head_dim, kv.page_size, reach, float(scale),
             _ptr(self.error_word), self._stream()), "paged_attention")
 
     # ---- latent attention, normalised adds, routed feed-forward ----------------------------------------------
@@ -1026,15 +1053,29 @@ class CudaKernels(KernelSet):
         else:
             raise KernelError(f"route_top: scores '{scores}' (chosen, all)")
 
+    def route_sigmoid(self, logits: torch.Tensor, experts: int, correction: Optional[torch.Tensor], groups, weight_scale: float,
+                      chosen: torch.Tensor, share: torch.Tensor) -> None:
+        """Scores s = sigmoid(logits[:, :experts]) (float32; further columns are not the router's); chosen[t] = the experts with
+        the largest s + `correction` (float32 [experts] or None), with `groups` = (count, keep) only among the `keep` of `count`
+        groups of neighbours whose two largest choice scores sum highest; share = weight_scale s / (sum of the chosen s + 1e-20)."""
+        T = logits.shape[0]
+        if logits.dtype != torch.float32 or (correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts)):
+            raise KernelError("route_sigmoid: float32 logits and one float32 correction per expert")
+        count, keep = groups if groups is not None else (0, 0)
+        self._count("route_sigmoid")
+        _check(self._moe.kvb_route_sigmoid(_ptr(logits), logits.shape[1], _ptr(correction), _ptr(chosen), _ptr(share), T, int(experts),
+                                           chosen.shape[1], int(count), int(keep), float(weight_scale), self._stream()), "route_sigmoid")
+
     ROUTED_SMALL_PAIRS = 256      # up to this many (row, choice) pairs the grouped products use tiles of 16 rows, else of 64
 
     def routed_experts(self, x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor,
                        share: torch.Tensor, out: torch.Tensor, activation: str, workspace, limit: float = 0.0,
-                       base: Optional[torch.Tensor] = None) -> None:
+                       base: Optional[torch.Tensor] = None, base_gate=None) -> None:
         """out[t] = base[t] + sum_s share[t, s] * w_down[e] . act(w_up[e] . x[t]), e = chosen[t, s]; w_down [E, H, F].
         "relu2": w_up [E, F, H], act = relu(.)^2.  "clamped_swiglu": w_up [E, 2 F, H] with gate row i at 2 i and up row i
         at 2 i + 1, act = g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).  "swiglu":
-        the same layout, act = silu(g) u (the kernels' gated epilogue with no limit)."""
+        the same layout, act = silu(g) u (the kernels' gated epilogue with no limit).  `base_gate` = (logits, col): base[t] is
+        multiplied by sigmoid(logits[t, col]) (float32)."""
         if activation not in ("relu2", "clamped_swiglu", "swiglu"):
             raise KernelError(f"routed_experts: activation '{activation}' is not built")
         if activation == "clamped_swiglu" and not limit > 0.0:
@@ -1044,7 +1085,7 @@ class CudaKernels(KernelSet):
         top = chosen.shape[1]
         if activation != "relu2" or base is not None:
             self._routed_general(x, w_up, w_down, chosen, share, out, 1 if activation == "relu2" else 2,
-                                 float(limit) if activation == "clamped_swiglu" else 0.0, base, workspace)
+                                 float(limit) if activation == "clamped_swiglu" else 0.0, base, workspace, base_gate)
             return
         pairs = T * top
         ws, i32 = workspace, torch.int32
@@ -1092,7 +1133,20 @@ class CudaKernels(KernelSet):
         self._count("routed_combine")
         _check(self._moe.kvb_routed_combine(code, _ptr(y), _ptr(place), _ptr(share), _ptr(out), T, top, H, stream), "routed_combine")
 
-    def _routed_general(self, x, w_up, w_down, chosen, share, out, act: int, limit: float, base, ws) -> None:
+    def _combine(self, code, y, place, share, base, base_gate, out, T, top, H, stream) -> None:
+        self._count("routed_combine")
+        if base_gate is None:
+            _check(self._moe.kvb_routed_combine_base(code, _ptr(y), _ptr(place), _ptr(share), _ptr(base), _ptr(out), T, top, H, stream),
+                   "routed_combine")
+            return
+        g, col = base_gate
+        if base is None or g.dtype != torch.float32 or g.shape[0] != T or not 0 <= col < g.shape[1]:
+            raise KernelError("routed_experts: the base's gate is one float32 logit per row of a base")
+        _ptr(g)                                                    # the checks of a device tensor
+        _check(self._moe.kvb_routed_combine_gated(code, _ptr(y), _ptr(place), _ptr(share), _ptr(base), _c_void_p(g.data_ptr() + 4 * col),
+                                                  g.shape[1], _ptr(out), T, top, H, stream), "routed_combine")
+
+    def _routed_general(self, x, w_up, w_down, chosen, share, out, act: int, limit: float, base, ws, base_gate=None) -> None:
         """The routed feed-forward with any of the grouped product's activations and an optional base: plan, product up
         (rows gathered, activation in the epilogue), product down, combine - float32 on CUDA cores, bfloat16 on `mma.sync`,
         and from `routed_tcgen05_min_pairs` pairs on through the tensor-memory kernel."""
@@ -1126,9 +1180,7 @@ class CudaKernels(KernelSet):
                 _check(self._gemm_grouped.kvb_grouped_gemm_tcgen05_act(_ptr(a), _ptr(w), _ptr(out_), _ptr(plan), _ptr(tiles), max_tiles,
                                                                        capacity, E, n, k, act_code, limit, _ptr(self.error_word),
                                                                        stream), f"grouped_gemm_tcgen05 ({what})")
-            self._count("routed_combine")
-            _check(self._moe.kvb_routed_combine_base(code, _ptr(y), _ptr(place), _ptr(share), _ptr(base), _ptr(out), T, top, H, stream),
-                   "routed_combine")
+            self._combine(code, y, place, share, base, base_gate, out, T, top, H, stream)
             return
         BM = 16 if pairs <= self.ROUTED_SMALL_PAIRS else 64
         max_tiles = -(-pairs // BM) + E
@@ -1144,9 +1196,7 @@ class CudaKernels(KernelSet):
         self._count("grouped_gemm")
         _check(self._moe.kvb_grouped_gemm_act(code, _ptr(hidden), _ptr(order), 0, _ptr(w_down), _ptr(y), _ptr(plan), _ptr(tiles),
                                               max_tiles, BM, H, F, 0, 0.0, stream), "grouped_gemm (down)")
-        self._count("routed_combine")
-        _check(self._moe.kvb_routed_combine_base(code, _ptr(y), _ptr(place), _ptr(share), _ptr(base), _ptr(out), T, top, H, stream),
-               "routed_combine")
+        self._combine(code, y, place, share, base, base_gate, out, T, top, H, stream)
 
     # ---- hashed pair embedding, gated heads, matrix-state mixers ---------------------------------------------
     def bigram_embed(self, table: torch.Tensor, batch: StepBatch, previous: torch.Tensor, h: torch.Tensor, buckets: int,

@@ -23,13 +23,14 @@ from ..parts.base import StepPlanner
 
 PREFILL_TILE_ROWS = 64          # query rows of a prefill attention tile
 PREFILL_KEY_TILE = 64           # keys the kernel takes at a time
+PREFILL_MIN_KEY_TILES = 4       # a unit has at least this many key tiles, unless its tile has fewer
 PREFILL_MAX_UNITS = 16          # most units one tile may be cut into (csrc/attention_flash.cu)
 PREFILL_UNITS_WANTED = 256      # about this many units beyond one per tile, however long the prompts
 TC_TILE_ROWS = 128              # query rows of a tile of the tensor-memory attention kernel
 TC_MIN_KEY_TILES = 16           # a unit of that kernel has at least this many key tiles, unless its tile has fewer
 
 
-def plan_prefill_units(segments, tile_rows: int = PREFILL_TILE_ROWS, min_key_tiles: int = 4):
+def plan_prefill_units(segments, tile_rows: int = PREFILL_TILE_ROWS, min_key_tiles: int = PREFILL_MIN_KEY_TILES):
     """`_plan_prefill_units`, remembered: a prompt cut into portions of one size, and prompts of one length, bring the
     same segments step after step.  The array that comes back is shared and not to be written."""
     return _plan_prefill_units(tuple(segments), tile_rows, min_key_tiles)

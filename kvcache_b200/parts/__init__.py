@@ -7,11 +7,11 @@ from .token_shift import TokenShiftMixer
 from .latent_attention import LatentAttention
 from .stream import LoopEntry
 from .model import CacheEntry, DecoderModel, LayerCall
-from .norm import RMSNorm
+from .norm import LayerNorm, RMSNorm
 from .position import NoPositionEncoding, RampScaling, RotaryHalf
 
 __all__ = ["GQAAttention", "Block", "FeedForward", "LayerContext", "Mixer", "Norm", "PagedKVSpec",
            "PagedKVView", "Part", "PositionEncoding", "Rotation", "StateSpec", "StepBatch", "StepPlan", "StepPlanner", "TORCH_DTYPES",
-           "PreNormBlock", "GatedMLP", "CacheEntry", "DecoderModel", "LayerCall", "RMSNorm",
+           "PreNormBlock", "GatedMLP", "CacheEntry", "DecoderModel", "LayerCall", "LayerNorm", "RMSNorm",
            "NoPositionEncoding", "RotaryHalf", "RampScaling", "SandwichBlock", "RoutedMLP", "LatentAttention", "LoopEntry",
            "ResidualGate", "ReluSquaredMLP", "TokenShiftMixer"]

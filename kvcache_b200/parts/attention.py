@@ -12,7 +12,8 @@ from typing import Dict, Mapping, Optional, Sequence
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import TORCH_DTYPES, LayerContext, Mixer, PagedKVSpec, PositionEncoding
+from .base import TORCH_DTYPES, BiasedDelta, LayerContext, Mixer, PagedKVSpec, PositionEncoding, reach_code
+from .position import interleaved_order
 
 
 class GQAAttention(Mixer):
@@ -34,7 +35,14 @@ class GQAAttention(Mixer):
     2^(-8 (h + 1) / H) (i - j) for a key i - j tokens back (after the cap, before the softmax).  `pad_values`: values
     narrower than keys are cached as wide as the keys, with zeros after their numbers, where that brings the layer to the
     tensor-core kernels, which take one size for both (bfloat16, keys of up to 128 numbers in steps of 16); the heads'
-    results then carry those zero columns, which the step after attention leaves out."""
+    results then carry those zero columns, which the step after attention leaves out.
+
+    `chunk`: a query sees the keys of its own chunk of this many tokens, counted from the request's first, up to itself (not
+    beside a window).  `rotary_layout` "interleaved": the rotation pairs neighbours (2 t, 2 t + 1) instead of dimensions half
+    the rotated ones apart; the rows of the projections are reordered when they are bound.  `out_bias`: the output matrix has
+    a bias, which is added with the delta (`forward` then returns a `BiasedDelta`).  `own_kv` False: the layer projects no
+    keys and values; its call reads the cache entry of another layer (which is told so: `keep_for`), with its own queries,
+    scale and mask."""
 
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, head_dim: int, *, qkv_bias: bool,
                  out_bias: bool, position: Optional[PositionEncoding], window: Optional[int], prefix: str,
@@ -44,16 +52,21 @@ class GQAAttention(Mixer):
                  qk_norm_scope: str = "head", qk_norm_weight: bool = True, qk_norm_after_rotation: bool = False,
                  sink=None, keep_first: int = 0, value_mix: Optional[str] = None, value_mix_name: str = "vmix",
                  q_temperature=None, score_cap: Optional[float] = None, distance_bias: Optional[str] = None,
-                 pad_values: bool = False):
+                 pad_values: bool = False, chunk: Optional[int] = None, rotary_layout: str = "half", own_kv: bool = True):
         if num_heads % num_kv_heads != 0:
             raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
-        if out_bias:
-            raise ValueError("an output-projection bias is not supported")
+        if rotary_layout not in ("half", "interleaved"):
+            raise ValueError(f"rotary_layout '{rotary_layout}' (half, interleaved)")
+        if not own_kv and value_mix is not None:
+            raise ValueError("a layer without values of its own cannot blend them")
         self.hidden, self.num_heads, self.num_kv_heads, self.head_dim = hidden, num_heads, num_kv_heads, head_dim
         self.value_dim = head_dim if value_dim is None else int(value_dim)
         self.qkv_bias = qkv_bias
         self.position = position
-        self.window = window
+        self.window, self.chunk = window, chunk
+        self.reach = reach_code(window, chunk)
+        self.cache_window, self.cache_chunk = window, chunk      # what the cache entry keeps: the widest of its readers' masks
+        self.out_bias, self.rotary_layout, self.own_kv = bool(out_bias), rotary_layout, bool(own_kv)
         self.prefix = prefix
         self.names = tuple(names)
         self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
@@ -86,7 +99,7 @@ class GQAAttention(Mixer):
         # The plain layer (equal key and value sizes, no norm of q and k, no gate) has fused and folded forms.
         self.plain = (self.value_dim == head_dim and self.qk_norm_eps is None and head_gate is None and sink is None
                       and not self.keep_first and value_mix is None and q_temperature is None and score_cap is None
-                      and distance_bias is None)
+                      and distance_bias is None and not out_bias and own_kv)
         # Keys narrower than values are cached as wide as the values, with zeros after their numbers (which add nothing
         # to a score), where that brings the layer to the tensor-core attention kernels, which take one size for both:
         # bfloat16, values of up to 128 numbers in steps of 16.  The cache then holds 2 value_dim numbers a token and
@@ -102,6 +115,7 @@ class GQAAttention(Mixer):
         self.w_qkv: Optional[torch.Tensor] = None
         self.b_qkv: Optional[torch.Tensor] = None
         self.w_o: Optional[torch.Tensor] = None
+        self.b_o: Optional[torch.Tensor] = None
         self.q_norm = self.k_norm = None
 
     def _bias_name(self, i: int) -> str:
@@ -113,18 +127,23 @@ class GQAAttention(Mixer):
         q, k, v, o = self.names
         specs = {
             p + q: TensorSpec((self.q_size, self.hidden)),
-            p + k: TensorSpec((self.kv_size, self.hidden)),
-            p + v: TensorSpec((self.v_size, self.hidden)),
             p + o: TensorSpec((self.hidden, self.heads_width)),
         }
+        if self.own_kv:
+            specs[p + k] = TensorSpec((self.kv_size, self.hidden))
+            specs[p + v] = TensorSpec((self.v_size, self.hidden))
         if self.qkv_bias:
             specs[self._bias_name(0)] = TensorSpec((self.q_size,))
-            specs[self._bias_name(1)] = TensorSpec((self.kv_size,))
-            specs[self._bias_name(2)] = TensorSpec((self.v_size,))
+            if self.own_kv:
+                specs[self._bias_name(1)] = TensorSpec((self.kv_size,))
+                specs[self._bias_name(2)] = TensorSpec((self.v_size,))
+        if self.out_bias:
+            specs[self._bias_name(3)] = TensorSpec((self.hidden,))
         if self.qk_norm_eps is not None and self.qk_norm_weight:
             whole = self.qk_norm_scope == "all"
             specs[p + q + ".norm"] = TensorSpec((self.q_size if whole else self.head_dim,))
-            specs[p + k + ".norm"] = TensorSpec((self.kv_size if whole else self.head_dim,))
+            if self.own_kv:
+                specs[p + k + ".norm"] = TensorSpec((self.kv_size if whole else self.head_dim,))
         if self.head_gate is not None:
             specs[p + self.head_gate] = TensorSpec((self.num_heads, self.hidden))
         if self.sink == "learned":
@@ -137,24 +156,46 @@ class GQAAttention(Mixer):
     def init_kinds(self) -> Dict[str, str]:
         if self.qk_norm_eps is None or not self.qk_norm_weight:
             return {}
-        return {self.prefix + self.names[0] + ".norm": "ones_plus_normal", self.prefix + self.names[1] + ".norm": "ones_plus_normal"}
+        return {self.prefix + name + ".norm": "ones_plus_normal" for name in (self.names[:2] if self.own_kv else self.names[:1])}
+
+    def keep_for(self, reader: "GQAAttention") -> None:
+        """`reader` reads this layer's cache entry: the entry keeps what either of them sees, and has the shape both expect."""
+        if self.keep_first or reader.keep_first:
+            raise ValueError("a cache entry with kept first keys is read by its own layer only")
+        reader.key_store, reader.value_store = self.key_store, self.value_store
+        if (reader.window, reader.chunk) == (self.cache_window, self.cache_chunk):
+            return
+        # A chunk's keys lie within a window of its size; so masks that differ are covered by a window of the widest.
+        sizes = [self.cache_window or self.cache_chunk, reader.window or reader.chunk]
+        self.cache_window, self.cache_chunk = (None if None in sizes else max(sizes)), None
+        self.plain = False                       # the fused forms take the cache entry's mask for the layer's
 
     def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
         p = self.prefix
+        # Queries and keys with their numbers in the order in which rotation partners lie half the rotated numbers apart.
+        order = torch.arange(self.head_dim)
+        if self.rotary_layout == "interleaved" and self.position is not None:
+            order = interleaved_order(self.head_dim, self.position.rotary_dim)
+        turned = lambda t: t if self.rotary_layout == "half" else \
+            t[(torch.arange(t.shape[0] // self.head_dim)[:, None] * self.head_dim + order[None, :]).reshape(-1)]
         # One projection for q, k and v (and the heads' gates): rows [q heads | k heads | v heads | gates].
-        rows = [tensors[p + n] for n in self.names[:3]]
+        parts = range(3) if self.own_kv else range(1)
+        rows = [tensors[p + self.names[i]] if i == 2 else turned(tensors[p + self.names[i]]) for i in parts]
         if self.head_gate is not None:
             rows.append(tensors[p + self.head_gate])
         self.w_qkv = torch.cat(rows, dim=0).to(self.dtype).to(device).contiguous()
         if self.qkv_bias:
-            bias = [tensors[self._bias_name(i)] for i in range(3)]
+            bias = [tensors[self._bias_name(i)] if i == 2 else turned(tensors[self._bias_name(i)]) for i in parts]
             if self.head_gate is not None:
                 bias.append(torch.zeros(self.num_heads))
             self.b_qkv = torch.cat(bias, dim=0).to(torch.float32).to(device).contiguous()
         self.w_o = tensors[p + self.names[3]].to(self.dtype).to(device).contiguous()
+        if self.out_bias:
+            self.b_o = tensors[self._bias_name(3)].to(torch.float32).to(device).contiguous()
         if self.qk_norm_eps is not None and self.qk_norm_weight:
-            self.q_norm = tensors[p + self.names[0] + ".norm"].to(torch.float32).to(device).contiguous()
-            self.k_norm = tensors[p + self.names[1] + ".norm"].to(torch.float32).to(device).contiguous()
+            self.q_norm = turned(tensors[p + self.names[0] + ".norm"]).to(torch.float32).to(device).contiguous()
+            if self.own_kv:
+                self.k_norm = turned(tensors[p + self.names[1] + ".norm"]).to(torch.float32).to(device).contiguous()
         if self.sink == "learned":
             self.sink_logits = tensors[p + "sink"].to(torch.float32).to(device).contiguous()
         elif self.sink is not None:
@@ -185,14 +226,16 @@ class GQAAttention(Mixer):
 
     def weight_bytes(self) -> int:
         n = self.w_qkv.numel() * self.w_qkv.element_size() + self.w_o.numel() * self.w_o.element_size()
-        return n + (self.b_qkv.numel() * 4 if self.b_qkv is not None else 0)
+        return n + sum(b.numel() * 4 for b in (self.b_qkv, self.b_o) if b is not None)
 
     def out_weight(self) -> torch.Tensor:
         return self.w_o
 
-    def cache_spec(self) -> PagedKVSpec:
-        return PagedKVSpec(self.num_kv_heads, self.key_store, self.window,
-                           None if self.value_store == self.key_store else self.value_store, self.keep_first)
+    def cache_spec(self) -> Optional[PagedKVSpec]:
+        if not self.own_kv:
+            return None
+        return PagedKVSpec(self.num_kv_heads, self.key_store, self.cache_window,
+                           None if self.value_store == self.key_store else self.value_store, self.keep_first, self.cache_chunk)
 
     def step_planners(self, kernels):
         planner = getattr(kernels, "paged_attention_planner", None)
@@ -223,6 +266,8 @@ class GQAAttention(Mixer):
         output matrix multiplies): the form a mixer that runs beside another one is asked for."""
         T = x.shape[0]
         k, ws = ctx.kernels, ctx.workspace
+        if ctx.kv.writes != self.own_kv:
+            raise ValueError("an attention layer writes the cache entry of its layer call exactly if it projects keys and values of its own")
         qkv = ws.buffer("attn.qkv", (T, self.w_qkv.shape[0]), self.dtype)
         k.linear(x, self.w_qkv, qkv)
         rotation = self.position.rotation() if self.position is not None else None
@@ -239,6 +284,8 @@ class GQAAttention(Mixer):
             extra["q_temperature"] = self.q_temperature
         if self.value_store != self.value_dim:
             extra["value_dim"] = self.value_dim
+        if not self.own_kv:
+            extra["queries_only"] = True
         k.qkv_rope_append(qkv, self.b_qkv, cos, sin, ctx.batch, ctx.kv, q, self.num_heads, q_norm=self.q_norm, k_norm=self.k_norm,
                           norm_eps=self.qk_norm_eps or 0.0, key_dim=self.head_dim, **extra)
         padded = self.value_store != self.value_dim
@@ -251,9 +298,11 @@ class GQAAttention(Mixer):
             more["score_cap"] = self.score_cap
         if self.slopes is not None:
             more["slopes"] = self.slopes
+        if self.reach != ctx.kv.spec.reach:
+            more["reach"] = self.reach                       # a cache entry that keeps more than this layer sees
         k.paged_attention(q, ctx.batch, ctx.kv, attn, self.num_heads, self.scale, ws, **more)
         if not direct:
-            gate = (qkv, self.q_size + self.kv_size + self.v_size) if self.head_gate is not None else None
+            gate = (qkv, self.q_size + (self.kv_size + self.v_size if self.own_kv else 0)) if self.head_gate is not None else None
             if padded:
                 k.head_gate(attn, gate, self.num_heads, self.value_dim, scale, out, out_col, x_head_stride=self.value_store)
             else:
@@ -267,7 +316,7 @@ class GQAAttention(Mixer):
             gated = ws.buffer("attn.gated", (T, self.heads_width), self.dtype)
             self.forward_heads(x, ctx, gated)
             k.linear(gated, self.w_o, delta)
-            return delta
+            return delta if self.b_o is None else BiasedDelta(delta, self.b_o)
         qkv = ws.buffer("attn.qkv", (T, self.q_size + 2 * self.kv_size), self.dtype)
         k.linear(x, self.w_qkv, qkv)
         rotation = self.position.rotation() if self.position is not None else None

@@ -28,11 +28,28 @@ from ..weights.loader import TensorSpec
 TORCH_DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32, "int32": torch.int32}
 
 
+def reach_code(window: Optional[int], chunk: Optional[int]) -> int:
+    """Which keys up to its own a query at position p sees, as one number: w > 0 - the last w (first key max(0, p - w + 1));
+    -c < 0 - those of its chunk of c tokens (first key p - p % c); 0 - all."""
+    if window is not None and chunk is not None:
+        raise ValueError("a layer has a window or chunks, not both")
+    return int(window) if window else -int(chunk) if chunk else 0
+
+
+def first_seen(position: int, reach: int) -> int:
+    """The first key that a query at `position` sees under `reach` (see `reach_code`)."""
+    if reach > 0:
+        return max(0, position - reach + 1)
+    return position - position % -reach if reach < 0 else 0
+
+
 @dataclass(frozen=True)
 class PagedKVSpec:
     """Pages of keys and values: `[pages, num_kv_heads, page_size, head_dim]` for K and for V.
 
     `window`: how many keys, its own included, a query sees (None: all of them).
+    `chunk`: a query sees the keys of its own chunk of this many tokens, counted from the request's first, up to itself
+    (None: no chunks; not beside a window).
     Layers whose specs are equal share a group: one block table, one page id
     for all of them, as the reference uses one table for its 24 layers
     (apps/qwen_serve.cu:99-100).
@@ -45,6 +62,12 @@ class PagedKVSpec:
     value_dim: Optional[int] = None
     # With a window: the request's first `keep_first` keys stay visible to every later query (and their pages stay held).
     keep_first: int = 0
+    chunk: Optional[int] = None
+
+    @property
+    def reach(self) -> int:
+        """Window and chunk as the kernels take them (see `reach_code`)."""
+        return reach_code(self.window, self.chunk)
 
     @property
     def v_head_dim(self) -> int:
@@ -155,6 +178,15 @@ class ScaledDelta:
     scale: torch.Tensor
 
 
+@dataclass
+class BiasedDelta:
+    """What a mixer or block hands on instead of a plain delta when its last product's bias is added together with the delta:
+    h += delta + bias (`bias` float32 [width], on the device), so that the bias is never rounded and costs no launch.
+    `Norm.add_norm` takes it wherever it takes a delta."""
+    delta: torch.Tensor
+    bias: torch.Tensor
+
+
 class Part:
     """Base of all parts: checkpoint tensors in, device buffers held."""
 
@@ -177,7 +209,7 @@ class Part:
 class Norm(Part):
     def add_norm(self, h: torch.Tensor, delta, out: Optional[torch.Tensor],
                  ctx: LayerContext, rows: Optional[torch.Tensor] = None, tail: Optional[torch.Tensor] = None) -> None:
-        """`delta`: None, a tensor, or a `NormedDelta` (normalised by its own norm before the add).  `out` None: only
+        """`delta`: None, a tensor, a `ScaledDelta`, a `BiasedDelta`, or a `NormedDelta` (normalised by its own norm before the add).  `out` None: only
         the add.  `tail` (float32 rows as wide as h): `out` has twice the width and its right half receives `tail`
         in the compute type, for a product over [normalised h | tail]."""
         raise NotImplementedError

@@ -7,7 +7,7 @@ from typing import Dict, Mapping, Optional
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import TORCH_DTYPES, Block, FeedForward, LayerContext, Mixer, Norm, Part, ScaledDelta
+from .base import TORCH_DTYPES, BiasedDelta, Block, FeedForward, LayerContext, Mixer, Norm, Part, ScaledDelta
 
 
 class LayerScale(Part):
@@ -88,6 +88,8 @@ class PreNormBlock(Block):
         self.norm1.add_norm(h, pending, x, ctx)
         delta = self.mixer.forward(x, ctx)
         if self.scale1 is not None:
+            if isinstance(delta, BiasedDelta):
+                raise ValueError("a mixer whose output has a bias cannot be scaled channel by channel before the add")
             delta = ScaledDelta(delta, self.scale1.scale)
         if self.ffn is None:
             return delta

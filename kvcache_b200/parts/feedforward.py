@@ -135,6 +135,12 @@ class RoutedMLP(FeedForward):
     feed-forward that every row takes, added to the routed sum.  `router_bias`: the name of a bias of the router's logits
     (one float32 number per expert), or None.
 
+    `scores` "sigmoid": scores s = sigmoid(logits); the choice goes by s + correction (`correction`: the name of one float32
+    number per expert, or None), the weights are `weight_scale` * s / (sum of the chosen s + 1e-20).  `groups` = (count, keep)
+    with these scores: the experts form `count` equal groups of neighbours, a group's value is the sum of its two largest
+    choice scores, and only experts of the `keep` groups with the largest values can be chosen.  `shared_gate`: the name of a
+    [1, hidden] matrix; the shared result is multiplied by sigmoid of that product, one number per row.
+
     The experts' matrices are stacked ([experts, ff, hidden] - gate and up rows in turn, [experts, 2 ff, hidden], for the
     gated form - and [experts, hidden, ff]) so that one grouped product serves all of them; which rows go to which expert
     is decided on the device, and the launches do not depend on it.
@@ -142,13 +148,20 @@ class RoutedMLP(FeedForward):
 
     def __init__(self, hidden: int, expert_ff: int, experts: int, top: int, *, activation: str, prefix: str, dtype: str,
                  router_name: str = "router", expert_names: Optional[Sequence[str]] = None, scores: str = "chosen",
-                 limit: float = 0.0, shared: Optional[FeedForward] = None, router_bias: Optional[str] = None):
+                 limit: float = 0.0, shared: Optional[FeedForward] = None, router_bias: Optional[str] = None,
+                 correction: Optional[str] = None, groups=None, weight_scale: float = 1.0, shared_gate: Optional[str] = None):
         if activation not in ROUTED_ACTIVATIONS:
             raise ValueError(f"activation '{activation}' is not supported by the routed feed-forward kernels")
         if not 1 <= top <= experts:
             raise ValueError(f"top {top} of {experts} experts")
-        if scores not in ("chosen", "all"):
-            raise ValueError(f"scores '{scores}' (chosen, all)")
+        if scores not in ("chosen", "all", "sigmoid"):
+            raise ValueError(f"scores '{scores}' (chosen, all, sigmoid)")
+        if scores != "sigmoid" and (correction is not None or groups is not None or weight_scale != 1.0):
+            raise ValueError("a correction, groups and a scale of the weights come with sigmoid scores")
+        if shared_gate is not None and (shared is None or scores != "sigmoid"):
+            raise ValueError("a gate of the shared feed-forward comes with one, and with sigmoid scores")
+        if groups is not None and (experts % groups[0] or not 1 <= groups[1] <= groups[0] or top > experts // groups[0] * groups[1]):
+            raise ValueError(f"groups {groups} of {experts} experts, {top} chosen")
         if activation == "clamped_swiglu" and not limit > 0.0:
             raise ValueError("the clamped activation needs a positive limit")
         self.hidden, self.expert_ff, self.experts, self.top = hidden, expert_ff, experts, top
@@ -156,6 +169,9 @@ class RoutedMLP(FeedForward):
         self.gated = activation in ("clamped_swiglu", "swiglu")
         self.router_bias = router_bias
         self.b_router: Optional[torch.Tensor] = None
+        self.correction_name, self.groups, self.weight_scale = correction, groups, float(weight_scale)
+        self.shared_gate = shared_gate
+        self.correction: Optional[torch.Tensor] = None
         if expert_names is None:
             expert_names = ("e{e}.gate", "e{e}.up", "e{e}.down") if self.gated else ("e{e}.up", "e{e}.down")
         if len(expert_names) != (3 if self.gated else 2):
@@ -176,6 +192,10 @@ class RoutedMLP(FeedForward):
         specs = {self.prefix + self.router_name: TensorSpec((self.experts, self.hidden))}
         if self.router_bias is not None:
             specs[self.prefix + self.router_bias] = TensorSpec((self.experts,))
+        if self.correction_name is not None:
+            specs[self.prefix + self.correction_name] = TensorSpec((self.experts,))
+        if self.shared_gate is not None:
+            specs[self.prefix + self.shared_gate] = TensorSpec((1, self.hidden))
         for e in range(self.experts):
             for which in range(len(self.expert_names) - 1):
                 specs[self._expert(which, e)] = TensorSpec((self.expert_ff, self.hidden))
@@ -190,9 +210,18 @@ class RoutedMLP(FeedForward):
     def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
         place = lambda t: t.to(self.dtype).to(device).contiguous()
         E = range(self.experts)
-        self.w_router = place(tensors[self.prefix + self.router_name])
+        router = [tensors[self.prefix + self.router_name]]
+        if self.shared_gate is not None:
+            # The shared feed-forward's gate is one more row of the router's product, zero rows after it up to a multiple of 8.
+            router.append(tensors[self.prefix + self.shared_gate])
+            if (self.experts + 1) % 8:
+                router.append(torch.zeros(8 - (self.experts + 1) % 8, self.hidden, dtype=router[0].dtype))
+        self.w_router = place(torch.cat(router, dim=0))
+        if self.correction_name is not None:
+            self.correction = tensors[self.prefix + self.correction_name].to(torch.float32).to(device).contiguous()
         if self.router_bias is not None:
-            self.b_router = tensors[self.prefix + self.router_bias].to(torch.float32).to(device).contiguous()
+            bias = tensors[self.prefix + self.router_bias].to(torch.float32)
+            self.b_router = torch.cat([bias, torch.zeros(self.w_router.shape[0] - self.experts)]).to(device).contiguous()
         if self.gated:
             # Row 2 i is gate row i, row 2 i + 1 up row i: a product's thread holds both numbers of an index.
             self.w_up = place(torch.stack([torch.stack([tensors[self._expert(0, e)], tensors[self._expert(1, e)]], dim=1)
@@ -214,7 +243,7 @@ class RoutedMLP(FeedForward):
         T = x.shape[0]
         k, ws = ctx.kernels, ctx.workspace
         base = self.shared.forward(x, ctx) if self.shared is not None else None
-        logits = ws.buffer("moe.logits", (T, self.experts), torch.float32)
+        logits = ws.buffer("moe.logits", (T, self.w_router.shape[0]), torch.float32)
         k.linear(x, self.w_router, logits, self.b_router)
         chosen = ws.buffer("moe.chosen", (T, self.top), torch.int32)
         share = ws.buffer("moe.share", (T, self.top), torch.float32)
@@ -222,6 +251,10 @@ class RoutedMLP(FeedForward):
         if self.scores == "chosen" and not self.gated and base is None:
             k.route_top(logits, chosen, share)
             k.routed_experts(x, self.w_up, self.w_down, chosen, share, delta, self.activation, ws)
+        elif self.scores == "sigmoid":
+            k.route_sigmoid(logits, self.experts, self.correction, self.groups, self.weight_scale, chosen, share)
+            extra = {} if self.shared_gate is None else {"base_gate": (logits, self.experts)}
+            k.routed_experts(x, self.w_up, self.w_down, chosen, share, delta, self.activation, ws, limit=self.limit, base=base, **extra)
         else:
             k.route_top(logits, chosen, share, scores=self.scores)
             k.routed_experts(x, self.w_up, self.w_down, chosen, share, delta, self.activation, ws, limit=self.limit, base=base)

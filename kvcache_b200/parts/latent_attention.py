@@ -34,6 +34,7 @@ import torch
 
 from ..weights.loader import TensorSpec
 from .base import TORCH_DTYPES, LayerContext, Mixer, PagedKVSpec, PositionEncoding
+from .position import interleaved_order
 
 
 class LatentAttention(Mixer):
@@ -101,7 +102,7 @@ class LatentAttention(Mixer):
             return torch.arange(self.rot_dim)
         rotation = self.position.rotation()
         dims = 2 * rotation.cos.shape[1] if rotation is not None else self.position.rotary_dim
-        return torch.cat([torch.arange(0, dims, 2), torch.arange(1, dims, 2), torch.arange(dims, self.rot_dim)])
+        return interleaved_order(self.rot_dim, dims)
 
     def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
         p, H = self.prefix, self.num_heads

@@ -6,7 +6,7 @@ from typing import Dict, Mapping, Optional
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import LayerContext, Norm, NormedDelta, ScaledDelta
+from .base import BiasedDelta, LayerContext, Norm, NormedDelta, ScaledDelta
 
 
 class RMSNorm(Norm):
@@ -42,6 +42,11 @@ class RMSNorm(Norm):
                 raise ValueError("a delta with a scale per channel is added by the launch that also normalises the rows")
             ctx.kernels.add_rmsnorm(h, delta.delta, self.weight, self.eps, out, rows, delta_scale=delta.scale)
             return
+        if isinstance(delta, BiasedDelta):
+            if out is None or tail is not None:
+                raise ValueError("a delta with a bias is added by the launch that also normalises the rows")
+            ctx.kernels.add_rmsnorm(h, delta.delta, self.weight, self.eps, out, rows, delta_bias=delta.bias)
+            return
         if isinstance(delta, NormedDelta) or out is None or tail is not None:
             # h += post.norm(delta), then this norm: one launch for both sums of squares.
             post = delta.post.fold_params() if isinstance(delta, NormedDelta) else None
@@ -57,6 +62,39 @@ class RMSNorm(Norm):
 
     def fold_params(self):
         return self.weight, self.eps
+
+
+class LayerNorm(Norm):
+    """y = (v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * weight, v = h + delta, in float32; the weight stays float32; no
+    bias.  It has no folded form (a product's rows would need their mean taken off first)."""
+
+    def __init__(self, width: int, eps: float, weight_name: str):
+        self.width = width
+        self.eps = float(eps)
+        self.weight_name = weight_name
+        self.weight: Optional[torch.Tensor] = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return {self.weight_name: TensorSpec((self.width,))}
+
+    def init_kinds(self) -> Dict[str, str]:
+        return {self.weight_name: "ones_plus_normal"}
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
+        self.weight = tensors[self.weight_name].to(torch.float32).to(device).contiguous()
+
+    def weight_bytes(self) -> int:
+        return self.width * 4
+
+    def add_norm(self, h, delta, out, ctx: LayerContext, rows=None, tail=None) -> None:
+        if out is None or tail is not None or isinstance(delta, NormedDelta):
+            raise ValueError("a centred norm takes plain, scaled and biased deltas and writes the normalised rows alone")
+        extra = {}
+        if isinstance(delta, ScaledDelta):
+            delta, extra["delta_scale"] = delta.delta, delta.scale
+        elif isinstance(delta, BiasedDelta):
+            delta, extra["delta_bias"] = delta.delta, delta.bias
+        ctx.kernels.add_rmsnorm(h, delta, self.weight, self.eps, out, rows, centred=True, **extra)
 
 
 class PassNorm(Norm):

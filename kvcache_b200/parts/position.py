@@ -98,5 +98,13 @@ class RotaryHalf(PositionEncoding):
         return self._rotation
 
 
+def interleaved_order(head_dim: int, rotary_dim: int) -> torch.Tensor:
+    """Where a head's numbers come from so that neighbours (2 t, 2 t + 1) of its first `rotary_dim` numbers end up `rotary_dim` / 2
+    apart: the even members, the odd members, then what is not rotated.  A score is a sum over a head's numbers and does not
+    change when queries and keys are reordered alike, so a projection whose rows are reordered once, when the weights are
+    bound, needs no rotation kernel of its own."""
+    return torch.cat([torch.arange(0, rotary_dim, 2), torch.arange(1, rotary_dim, 2), torch.arange(rotary_dim, head_dim)])
+
+
 class NoPositionEncoding(PositionEncoding):
     pass

@@ -5,6 +5,7 @@ run in tests on a machine without a GPU.  It is test code: the package has no CP
 """
 from __future__ import annotations
 
+import dataclasses
 from typing import Optional
 
 import torch
@@ -29,8 +30,10 @@ class TorchKernels:
             ids = torch.where(src >= 0, last[src.clamp(min=0).long()].long(), ids)
         out.copy_(table[ids].to(torch.float32) * scale)
 
-    def add_rmsnorm(self, h, delta, weight, eps, out, rows=None, delta_scale=None):
+    def add_rmsnorm(self, h, delta, weight, eps, out, rows=None, delta_scale=None, delta_bias=None, centred=False):
         f = self.f
+        if delta is not None and delta_bias is not None:
+            delta = delta.to(torch.float32) + delta_bias
         if delta is not None and delta_scale is not None:
             delta = delta.to(torch.float32) * delta_scale
         if rows is None:
@@ -41,6 +44,8 @@ class TorchKernels:
             v = h[rows.long()].to(f)
             if delta is not None:
                 v = (h[rows.long()] + delta[rows.long()].to(torch.float32)).to(f)
+        if centred:
+            v = v - v.mean(dim=-1, keepdim=True)
         inv = torch.rsqrt((v * v).mean(dim=-1, keepdim=True) + eps)
         out.copy_((v * inv * weight.to(f)).to(out.dtype))
 
@@ -51,9 +56,17 @@ class TorchKernels:
         out.copy_(y.to(out.dtype))
 
     def qkv_rope_append(self, qkv, bias, cos, sin, batch, kv, q_out, num_heads, q_norm=None, k_norm=None, norm_eps=0.0, key_dim=None,
-                        norm_scope="head", norm_after_rotation=False, value_mix=None, q_temperature=None, value_dim=None):
+                        norm_scope="head", norm_after_rotation=False, value_mix=None, q_temperature=None, value_dim=None,
+                        queries_only=False):
         f = self.f
         T = qkv.shape[0]
+        if queries_only:                  # rows of `num_heads` queries and nothing to append: as if there were no keys and values
+            assert not kv.writes
+            wide = kv.spec.head_dim - (key_dim or kv.spec.head_dim)
+            x = qkv.to(f) if bias is None else qkv.to(f) + bias.to(f)
+            none = dataclasses.replace(kv, spec=dataclasses.replace(kv.spec, num_kv_heads=0))
+            return self._qkv_norm_rope_append(x, cos, sin, batch, none, q_out, num_heads, q_norm, None, norm_eps, kv.spec.head_dim - wide,
+                                              norm_scope, norm_after_rotation, None, q_temperature, value_dim)
         Hq, Hkv, D = num_heads, kv.spec.num_kv_heads, kv.spec.head_dim
         x = qkv.to(f)
         if bias is not None:
@@ -103,6 +116,8 @@ class TorchKernels:
                 v = (1.0 - lam.to(f)) * v + lam.to(f) * kept.to(f).view(T, Hkv, Dv)
 
         def normalise(t, weight):
+            if t.shape[1] == 0:
+                return t
             if scope == "all":
                 flat = t.reshape(T, -1)
                 flat = flat * torch.rsqrt((flat * flat).mean(dim=-1, keepdim=True) + eps)
@@ -137,22 +152,23 @@ class TorchKernels:
             kv.k_pages[page, :, pos % kv.page_size, :] = k.to(kv.k_pages.dtype)
             kv.v_pages[page, :, pos % kv.page_size, :] = v.to(kv.v_pages.dtype)
 
-    def paged_attention(self, q, batch, kv, out, num_heads, scale, workspace=None, sink=None, score_cap=None, slopes=None):
+    def paged_attention(self, q, batch, kv, out, num_heads, scale, workspace=None, sink=None, score_cap=None, slopes=None, reach=None):
         """`sink` [Hq]: the softmax's denominator also holds exp(sink[h]).  kv.spec.keep_first: with a window, the
-        request's first keys stay visible.  `score_cap`: s <- cap tanh(s / cap); `slopes` [Hq]: s <- s - slopes[h] (i - j)."""
+        request's first keys stay visible.  `reach` (None: the cache entry's own): w > 0 a window, -c < 0 chunks of c tokens,
+        0 all keys.  `score_cap`: s <- cap tanh(s / cap); `slopes` [Hq]: s <- s - slopes[h] (i - j)."""
         f = self.f
         T = q.shape[0]
         Hq, Hkv, D = num_heads, kv.spec.num_kv_heads, kv.spec.head_dim
         group = Hq // Hkv
-        window = kv.spec.window
+        reach = kv.spec.reach if reach is None else reach
         qf = q.to(f).view(T, Hq, D)
         result = torch.zeros(T, Hq, kv.spec.v_head_dim, dtype=f, device=q.device)
         for r in range(T):
             p = int(batch.positions[r])
             seg = int(batch.row_segment[r])
-            lo = max(0, p - window + 1) if window else 0
+            lo = max(0, p - reach + 1) if reach > 0 else p // -reach * -reach if reach < 0 else 0
             js = torch.arange(lo, p + 1, device=q.device)
-            if window and kv.spec.keep_first:
+            if reach > 0 and kv.spec.keep_first:
                 js = torch.cat([torch.arange(0, min(lo, kv.spec.keep_first), device=q.device), js])
             pages = kv.block_table[seg, js // kv.page_size].long()
             assert bool((pages >= 0).all()), "a needed key lies in a page the block table does not hold"
@@ -310,9 +326,27 @@ class TorchKernels:
         else:
             share.copy_(torch.softmax(best, dim=-1).to(torch.float32))
 
-    def routed_experts(self, x, w_up, w_down, chosen, share, out, activation, workspace=None, limit=0.0, base=None):
+    def route_sigmoid(self, logits, experts, correction, groups, weight_scale, chosen, share):
+        """Scores s = sigmoid(logits[:, :experts]); the choice by s + correction, within the `keep` of `count` groups whose two
+        largest choice scores sum highest; share = weight_scale s / (sum of the chosen s + 1e-20)."""
+        s = torch.sigmoid(logits[:, :experts].to(self.f))
+        c = s if correction is None else s + correction.to(self.f)
+        if groups is not None:
+            count, keep = groups
+            split = c.view(c.shape[0], count, experts // count)
+            value = torch.topk(split, min(2, experts // count), dim=-1).values.sum(dim=-1)
+            out = torch.ones_like(value, dtype=torch.bool).scatter(1, torch.topk(value, keep, dim=-1).indices, False)
+            c = split.masked_fill(out[:, :, None], -torch.inf).reshape(c.shape)
+        which = torch.topk(c, chosen.shape[1], dim=-1).indices
+        chosen.copy_(which.to(torch.int32))
+        taken = torch.gather(s, 1, which)
+        share.copy_((taken / (taken.sum(dim=-1, keepdim=True) + 1e-20) * weight_scale).to(torch.float32))
+
+    def routed_experts(self, x, w_up, w_down, chosen, share, out, activation, workspace=None, limit=0.0, base=None, base_gate=None):
         f = self.f
         result = torch.zeros(x.shape[0], w_down.shape[1], dtype=f) if base is None else base.to(f).clone()
+        if base_gate is not None:                 # (logits, column): the base times sigmoid of that column
+            result = result * torch.sigmoid(base_gate[0][:, base_gate[1]].to(f))[:, None]
         for r in range(x.shape[0]):
             for s in range(chosen.shape[1]):
                 e = int(chosen[r, s])
