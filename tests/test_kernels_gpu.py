@@ -549,9 +549,9 @@ def test_paged_attention_tc(kernels, request, scenario):
         for i, (cached, new) in enumerate(segments):
             gone = max(0, cached - window + 1) // page
             kv.block_table[i, :gone] = -1
-    saved = kernels.tc_attention_min_rows
-    kernels.tc_attention_min_rows = 2
-    request.addfinalizer(lambda: setattr(kernels, "tc_attention_min_rows", saved))
+    saved, saved_min = kernels.tc_attention_min_rows, kernels.tc_unit_min_tiles
+    kernels.tc_attention_min_rows, kernels.tc_unit_min_tiles = 2, 1
+    request.addfinalizer(lambda: (setattr(kernels, "tc_attention_min_rows", saved), setattr(kernels, "tc_unit_min_tiles", saved_min)))
     ws = Workspace(DEV)
     rows = torch.arange(T)                                    # every row: segments of one row go through the decode kernel
     for _ in range(2):                                        # twice: the tickets of the first call must be zero again
@@ -570,9 +570,9 @@ def test_paged_attention_random_shapes(kernels, request, seed):
     import random
     from kvcache_b200.engine.workspace import Workspace
     rng = random.Random(seed)
-    saved = kernels.tc_attention_min_rows
-    kernels.tc_attention_min_rows = 2
-    request.addfinalizer(lambda: setattr(kernels, "tc_attention_min_rows", saved))
+    saved, saved_min = kernels.tc_attention_min_rows, kernels.tc_unit_min_tiles
+    kernels.tc_attention_min_rows, kernels.tc_unit_min_tiles = 2, 1
+    request.addfinalizer(lambda: (setattr(kernels, "tc_attention_min_rows", saved), setattr(kernels, "tc_unit_min_tiles", saved_min)))
     ws = Workspace(DEV)
     for it in range(8):
         D, Hkv, G = rng.choice([64, 128]), rng.choice([1, 2, 4]), rng.choice([1, 2, 3, 7])

@@ -231,6 +231,7 @@ def test_tensor_core_attention_with_a_sink_and_kept_first_keys(kernels, path, Hq
             k.tc_attention_min_rows, k.decode_merge = None, "ticket"
         else:
             k.tc_attention_min_rows, min_tiles = 128, 2
+            k.tc_unit_min_tiles = min_tiles
     dtype = torch.bfloat16
     batch, kv = paged_scenario([(0, 700), (2500, 1), (1500, 300), (900, 1), (63, 1), (0, 1), (3, 2), (1100, 130)], num_kv_heads=Hkv, head_dim=D,
                                page_size=16, dtype=dtype, device="cpu", seed=11, window=window, tc_min_key_tiles=min_tiles)
