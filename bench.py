@@ -1,7 +1,7 @@
 """Benchmark of kvcache_b200: decode tokens a second of the Qwen2.5-0.5B shape on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-    python bench.py --design kakipel|libulorn|lipelix|karorax [--sizes 0.5B-like,3B-like]     (another workload, see `run_design`; the default stays as it is)
+    python bench.py --design kakipel|libulorn|lipelix|karorax|kunulorn [--sizes 0.5B-like,3B-like]     (another workload, see `run_design`; the default stays as it is)
 
 One JSON line on standard output.  `value`: decoded tokens a second at batch 8 and the
 benchmark context (device-timed decode steps through the engine's step function and device
@@ -521,6 +521,32 @@ def karorax_sizes():
     return out
 
 
+def kunulorn_sizes():
+    """Layer sizes that resemble real models, as (name, {architecture: config}): a Kunulorn model of four layers (attention in
+    chunks of 1,024 tokens with the dense clamped feed-forward; the same with a routed feed-forward whose chosen experts and
+    shared expert together have as many active weights per token as the dense one; then both feed-forwards once more behind
+    attention that reads the first layer's keys and values), beside the Libulorn, Lipelix and Qwen2 models of `lipelix_sizes` at
+    equal width, heads, feed-forward width and vocabulary: Libulorn has the closest routed feed-forward and attention over
+    as many keys (a window of 1,024), Lipelix the norm over whole projections, Qwen2 the plain layer."""
+    out = []
+    others = dict(lipelix_sizes())
+    for name, width, heads, kv_heads, dim, ff, experts, top, vocab in (
+            ("0.5B-like", 896, 14, 2, 64, 4864, 16, 2, 32768),
+            ("3B-like", 2048, 16, 2, 128, 11008, 32, 4, 32768)):
+        own = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": 1024},
+               "rot": {"base": 500000.0, "dims": dim // 2}}
+        read = dict(own, kv_from=0)
+        dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+        moe = {"kind": "moe", "expert": {"ff": ff // (2 * top) // 16 * 16}, "shared": {"ff": ff // 2},
+               "router": {"experts": experts, "top": top, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+        kun = {"architecture": "Kunulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+               "layers": [{"type": "attention", "mixer": m, "mlp": f} for m, f in ((own, dense), (own, moe), (read, dense), (read, moe))],
+               "initializer_range": 0.02}
+        out.append((name, {"kunulorn": kun, "libulorn": others[name]["libulorn"], "lipelix": others[name]["lipelix"],
+                           "qwen2": others[name]["qwen2"]}))
+    return out
+
+
 def _write_design_folder(tmp, tag, config):
     import torch
     import kvcache_b200  # noqa: F401
@@ -613,7 +639,7 @@ def _time_classes(folder, peaks, mode, batch, context, tokens, repeats=3):
 
 
 def run_design(args) -> int:
-    """`--design kakipel | libulorn | lipelix | karorax`: decode and prefill throughput of that architecture at sizes that resemble real models'
+    """`--design kakipel | libulorn | lipelix | karorax | kunulorn`: decode and prefill throughput of that architecture at sizes that resemble real models'
     layers, beside the Qwen2 architecture at equal width, layer runs, feed-forward width and vocabulary (random weights,
     random cache contents for decode), and every class of kernel of one step of each against its roofline."""
     peaks = load_peaks()
@@ -625,6 +651,8 @@ def run_design(args) -> int:
         sizes, beside = lipelix_sizes(), "Lipelix beside Libulorn and Qwen2"
     elif args.design == "karorax":
         sizes, beside = karorax_sizes(), "Karorax beside Libulorn, Kakipel and Qwen2"
+    elif args.design == "kunulorn":
+        sizes, beside = kunulorn_sizes(), "Kunulorn beside Libulorn, Lipelix and Qwen2"
     else:
         sizes, beside = [(name, {"kakipel": kaki, "qwen2": qwen}) for name, kaki, qwen in design_sizes()], "Kakipel beside Qwen2"
     done = {}
@@ -747,7 +775,7 @@ def main() -> int:
     parser.add_argument("--skip-prefill", action="store_true")
     parser.add_argument("--skip-kernels", action="store_true")
     parser.add_argument("--no-graphs", action="store_true", help="launch the decode step's kernels one by one (for profilers)")
-    parser.add_argument("--design", default=None, choices=["kakipel", "libulorn", "lipelix", "karorax"],
+    parser.add_argument("--design", default=None, choices=["kakipel", "libulorn", "lipelix", "karorax", "kunulorn"],
                         help="instead of the default workload: this architecture beside Qwen2 at equal sizes (decode, prefill, kernels)")
     parser.add_argument("--sizes", default="", help="with --design: the sizes to run, with commas between them (default: all)")
     args = parser.parse_args()

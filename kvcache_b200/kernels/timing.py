@@ -24,20 +24,21 @@ from typing import Callable, Dict, List, Tuple
 
 import torch
 
+from ..parts.base import first_seen
+
 
 def _numel_bytes(t) -> int:
     return 0 if t is None else t.numel() * t.element_size()
 
 
-def _attention_bytes(batch, kv, num_heads: int) -> int:
-    """Keys and values of the step's requests (every key once per kv head), queries in, results out."""
+def _attention_bytes(batch, kv, num_heads: int, reach=None) -> int:
+    """Keys and values of the step's requests (every key that a row sees, once per kv head), queries in, results out."""
     spec = kv.spec
+    reach = spec.reach if reach is None else reach
     element = kv.k_pages.element_size()
     host = batch.host
     if "starts" in host and "counts" in host:
-        keys = int((host["starts"] + host["counts"]).sum())
-        if spec.window:
-            keys = int(sum(min(int(s + c), spec.window + int(c) - 1) for s, c in zip(host["starts"], host["counts"])))
+        keys = int(sum(int(s + c) - first_seen(int(s), reach) for s, c in zip(host["starts"], host["counts"])))
     else:
         keys = batch.max_kv_len * batch.num_segments
     rows = batch.num_tokens * num_heads * spec.head_dim * element
@@ -47,7 +48,7 @@ def _attention_bytes(batch, kv, num_heads: int) -> int:
 class KernelTiming:
     OPERATORS = ("embed", "add_rmsnorm", "silu_mul", "gate_up_act", "linear", "qkv_rope_append", "rope_append_attention",
                  "paged_attention", "sample", "norm_add_rmsnorm", "latent_norm_rope_append", "head_linear", "latent_attention",
-                 "route_top", "routed_experts", "bigram_embed", "head_gate", "head_norm_gate", "gated_linear_scan",
+                 "route_top", "route_sigmoid", "routed_experts", "bigram_embed", "head_gate", "head_norm_gate", "gated_linear_scan",
                  "matrix_memory_scan", "token_shift", "activation_", "delta_rule_scan", "lightning_scan")
 
     def __init__(self, kernels, hold_ms: float = 4.0):
@@ -82,7 +83,7 @@ class KernelTiming:
             return name, _attention_bytes(batch, kv, num_heads) + _numel_bytes(qkv)
         if name == "paged_attention":
             batch, kv, num_heads = args[1], args[2], args[4]
-            return name, _attention_bytes(batch, kv, num_heads)
+            return name, _attention_bytes(batch, kv, num_heads, kwargs.get("reach"))
         if name == "sample":
             return name, _numel_bytes(args[0])
         if name == "norm_add_rmsnorm":
@@ -103,7 +104,7 @@ class KernelTiming:
             if window and "starts" in host:
                 keys = int(sum(min(int(s + c), window + int(c) - 1) for s, c in zip(host["starts"], host["counts"])))
             return name, keys * kv.spec.head_dim * kv.k_pages.element_size() + _numel_bytes(q) + _numel_bytes(out)
-        if name == "route_top":
+        if name in ("route_top", "route_sigmoid"):
             return name, _numel_bytes(args[0])
         if name == "routed_experts":
             x, w_up, w_down, chosen, out = args[0], args[1], args[2], args[3], args[5]
@@ -143,19 +144,19 @@ class KernelTiming:
         return name, 0
 
     @staticmethod
-    def _keys_seen(batch, spec=None) -> int:
-        """Sum over the step's rows of the keys a row sees (its own included): all up to its position, or with a window
-        the window's keys and the kept first ones behind it."""
+    def _keys_seen(batch, reach: int = 0, keep: int = 0) -> int:
+        """Sum over the step's rows of the keys a row sees (its own included): all up to its position, or those of its window
+        (and the kept first ones behind it) or chunk."""
         host = batch.host
         if "starts" not in host:
             return batch.num_tokens * batch.max_kv_len
-        window = getattr(spec, "window", None)
-        if not window:
+        if not reach:
             return int(sum(int(c) * int(s) + int(c) * (int(c) + 1) // 2 for s, c in zip(host["starts"], host["counts"])))
-        keep, total = int(getattr(spec, "keep_first", 0) or 0), 0
+        total = 0
         for s, c in zip(host["starts"], host["counts"]):
             for p in range(int(s), int(s) + int(c)):
-                total += min(p + 1, window) + max(0, min(keep, p + 1 - window))
+                lo = first_seen(p, reach)
+                total += p + 1 - lo + (min(keep, lo) if reach > 0 else 0)
         return total
 
     @classmethod
@@ -171,18 +172,14 @@ class KernelTiming:
         if name == "latent_attention":
             batch, kv, heads, value_dim = args[1], args[2], args[4], args[5]
             window = kwargs.get("window", -1)
-
-            class _Reach:
-                pass
-            reach = _Reach()
-            reach.window, reach.keep_first = (kv.spec.window if window == -1 else window), 0
-            return 2 * heads * (kv.spec.head_dim + value_dim) * cls._keys_seen(batch, reach)
+            return 2 * heads * (kv.spec.head_dim + value_dim) * cls._keys_seen(batch, (kv.spec.window if window == -1 else window) or 0)
         if name == "paged_attention":
             batch, kv, heads = args[1], args[2], args[4]
-            return 2 * heads * (kv.spec.head_dim + kv.spec.v_head_dim) * cls._keys_seen(batch, kv.spec)
+            reach = kwargs.get("reach")
+            return 2 * heads * (kv.spec.head_dim + kv.spec.v_head_dim) * cls._keys_seen(batch, kv.spec.reach if reach is None else reach, kv.spec.keep_first)
         if name == "rope_append_attention":
             batch, kv, heads = args[4], args[5], args[7]
-            return 2 * heads * (kv.spec.head_dim + kv.spec.v_head_dim) * cls._keys_seen(batch, kv.spec)
+            return 2 * heads * (kv.spec.head_dim + kv.spec.v_head_dim) * cls._keys_seen(batch, kv.spec.reach, kv.spec.keep_first)
         if name == "routed_experts":
             x, w_up, w_down, chosen = args[0], args[1], args[2], args[3]
             return 2 * chosen.numel() * (w_up.shape[1] * w_up.shape[2] + w_down.shape[1] * w_down.shape[2])
