@@ -20,7 +20,7 @@ import sys
 from typing import Dict
 
 PAGE_SIZE = 16          # default of --page-size; divides 64, the rounding of --max-tokens
-MAX_LIVE_REQUESTS = 8   # default of --max-live
+MAX_LIVE_REQUESTS = 4   # default of --max-live
 
 
 def main(argv=None) -> int:

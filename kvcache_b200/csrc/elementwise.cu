@@ -509,29 +509,59 @@ KVB_API int kvb_token_shift(int dtype, const void* x, const float* w, float* pre
     return kvb_launch_status();
 }
 
-// x = act(x) in place; kind 0: tanh, 1: relu(x)^2, 2: cap * tanh(x / cap).
-template <typename T>
-__global__ void activation_kernel(T* __restrict__ x, size_t total, int kind, float cap) {
+// out[t, out_col + i] = act(x[t, i]); kind 0: tanh, 1: relu(x)^2, 2: cap * tanh(x / cap), 3: x Phi(x) with the normal distribution
+// function (the exact gelu).  x: rows of x_stride, `cols` of them taken from x_col on; out may be x itself.  A thread takes VEC
+// neighbouring numbers of a row.
+__device__ __forceinline__ float activate(float v, int kind, float cap) {
+    if (kind == 0) return tanhf(v);
+    if (kind == 1) { const float p = fmaxf(v, 0.f); return p * p; }
+    if (kind == 2) return cap * tanhf(v / cap);
+    return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+}
+
+template <typename T, int VEC>
+__global__ void activation_kernel(const T* x, int x_stride, int x_col, T* out, int out_stride, int out_col, int per_row, long long total,
+                                  int kind, float cap) {
     pdl_wait();
     pdl_launch_dependents();
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-        const float v = to_f32<T>(x[i]);
-        const float p = fmaxf(v, 0.f);
-        x[i] = from_f32<T>(kind == 0 ? tanhf(v) : kind == 1 ? p * p : cap * tanhf(v / cap));
+    struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
+    for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (long long)gridDim.x * blockDim.x) {
+        const long long t = total <= 0x7fffffffLL ? (long long)((int)idx / per_row) : idx / per_row;
+        const int c = (int)(idx - t * per_row) * VEC;
+        Pack p = *reinterpret_cast<const Pack*>(x + t * x_stride + x_col + c);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(activate(to_f32<T>(p.v[e]), kind, cap));
+        *reinterpret_cast<Pack*>(out + t * out_stride + out_col + c) = p;
     }
 }
 
-KVB_API int kvb_activation(int dtype, void* x, long long total, int kind, float cap, cudaStream_t stream) {
-    if (total <= 0) return KVB_OK;
-    if (kind < 0 || kind > 2 || (kind == 2 && !(cap > 0.f))) return KVB_ERR_SHAPE;
-    long long blocks = (total + 255) / 256;
-    const long long most = (long long)kvb_sm_count() * 16;
+template <typename T>
+static int launch_activation(const T* x, int x_stride, int x_col, T* out, int out_stride, int out_col, long long T_, int cols, int kind,
+                             float cap, cudaStream_t stream) {
+    constexpr int V = 16 / (int)sizeof(T);
+    const bool wide = ((cols | x_stride | x_col | out_stride | out_col) % V) == 0 && ((((uintptr_t)x) | ((uintptr_t)out)) & 15) == 0;
+    const int per_row = wide ? cols / V : cols;
+    const long long total = T_ * per_row;
+    long long blocks = (total + 127) / 128;
+    const long long most = (long long)kvb_sm_count() * 32;
     if (blocks > most) blocks = most;
-    if (dtype == KVB_F32)
-        kvb_launch(activation_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (float*)x, (size_t)total, kind, cap);
-    else if (dtype == KVB_BF16)
-        kvb_launch(activation_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, (bf16*)x, (size_t)total, kind, cap);
+    if (wide)
+        kvb_launch(activation_kernel<T, V>, dim3((unsigned)blocks), dim3(128), 0, stream, x, x_stride, x_col, out, out_stride, out_col, per_row,
+                   total, kind, cap);
     else
-        return KVB_ERR_DTYPE;
+        kvb_launch(activation_kernel<T, 1>, dim3((unsigned)blocks), dim3(128), 0, stream, x, x_stride, x_col, out, out_stride, out_col, per_row,
+                   total, kind, cap);
     return kvb_launch_status();
+}
+
+KVB_API int kvb_activation(int dtype, const void* x, int x_stride, int x_col, void* out, int out_stride, int out_col, long long T, int cols,
+                           int kind, float cap, cudaStream_t stream) {
+    if (T <= 0 || cols <= 0) return KVB_OK;
+    if (kind < 0 || kind > 3 || (kind == 2 && !(cap > 0.f)) || x_col < 0 || out_col < 0 || x_col + cols > x_stride || out_col + cols > out_stride)
+        return KVB_ERR_SHAPE;
+    if (dtype == KVB_F32)
+        return launch_activation<float>((const float*)x, x_stride, x_col, (float*)out, out_stride, out_col, T, cols, kind, cap, stream);
+    if (dtype == KVB_BF16)
+        return launch_activation<bf16>((const bf16*)x, x_stride, x_col, (bf16*)out, out_stride, out_col, T, cols, kind, cap, stream);
+    return KVB_ERR_DTYPE;
 }

@@ -3,8 +3,12 @@
 //
 //   matrix_state_scan   S_t = decay_t S_{t-1} + gain_t k_t v_t^T, o_t = S_t^T q_t over the tokens of every segment, from
 //                       and into the request's state slot; two forms of decay (below)
+//   short convolutions  causal, per channel, over the last few tokens, with what the delta rule or the state space reads made in
+//                       the same launch (unit vectors, decays, step sizes); the last inputs of a request are its state
+//   gated_delta_scan    S~ = diag(a) S, S' = S~ + k (b (v - S~^T k))^T, o = S'^T q
+//   state_space_scan    S' = exp(-A d) S + d B x^T, o = S'^T C, and what follows it (gate, norm over parts of a row)
 //   head_norm_gate      out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * act(gate[t, h, :]) * scale
-//   head_gate           out[t, h, :] = x[t, h, :] * sigmoid(gate[t, h]) * scale
+//   head_gate           out[t, h, :] = x[t, h, :] * sigmoid(gate[t, h]) * scale, or with a gate per channel
 //   bigram_embed        h[r] += table[(previous token * a + token * b) mod buckets], the table's last row at position 0;
 //                       then the request's previous token becomes the last one of its segment
 //
@@ -27,7 +31,7 @@
 // slot.  The arithmetic per token is the same as in one piece; the start states differ from it by float32 rounding.
 #include "common.cuh"
 
-enum { SCAN_CHANNEL_DECAY = 0, SCAN_EXP_GATES = 1, SCAN_DELTA_RULE = 2 };
+enum { SCAN_CHANNEL_DECAY = 0, SCAN_EXP_GATES = 1, SCAN_DELTA_RULE = 2, SCAN_GATED_DELTA = 3, SCAN_HEAD_DECAY = 4 };
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
@@ -43,12 +47,12 @@ struct ScanChunks {
     int L, S;              // tokens in a chunk; segments in the step
     float* local_S;        // [chunk, H, D, Dv]   end state of the chunk scanned from an empty state
     float* local_vec;      // [chunk, H, D]       channel decay: the product of the chunk's decays; exponential gates: its normaliser
-    float* local_F;        // [chunk, H]          exponential gates: the sum of the chunk's log forget gates
+    float* local_F;        // [chunk, H]          exponential gates: the sum of the chunk's log forget gates; head decay: the product of its decays
     float* local_m;        // [chunk, H]          exponential gates: the chunk's maximum from an empty state
     float* start_S;        // [chunk, H, D, Dv]   state before the chunk's first token
     float* start_vec;      // [chunk, H, D]       exponential gates: the normaliser there
     float* start_m;        // [chunk, H]          exponential gates: the maximum there
-    float* local_P;        // [chunk, H, D, D]    delta rule: the chunk's transition, the product of its tokens' diag(w) - (a u) u^T
+    float* local_P;        // [chunk, H, D, D]    delta rules: the chunk's transition, the product of its tokens' diag(w) - (a u) u^T
 };
 
 // Which (segment, chunk of it) the chunk id is; false beyond the step's last chunk.
@@ -68,8 +72,14 @@ __device__ __forceinline__ bool find_chunk(int id, const ScanChunks& ch, const i
 enum { SCAN_LOCAL = 1, SCAN_FROM_START = 3 };
 constexpr int SCAN_TILE = 32;          // tokens staged at a time
 // Rows of key channels staged per token (q, k, then the mode's own), and the tokens staged at a time: the delta rule
-// stages five rows a token and takes half the tokens, so that heads of 256 key channels still fit.
-__host__ __device__ constexpr int scan_parts(int mode) { return mode == SCAN_CHANNEL_DECAY ? 3 : mode == SCAN_DELTA_RULE ? 5 : 2; }
+// stages five rows a token and takes half the tokens, so that heads of 256 key channels still fit.  After them come the
+// mode's numbers per token and head (scan_scalars).
+__host__ __device__ constexpr int scan_parts(int mode) {
+    return mode == SCAN_CHANNEL_DECAY || mode == SCAN_GATED_DELTA ? 3 : mode == SCAN_DELTA_RULE ? 5 : 2;
+}
+__host__ __device__ constexpr int scan_scalars(int mode) { return mode == SCAN_GATED_DELTA ? 1 : mode == SCAN_HEAD_DECAY ? 2 : 0; }
+// Forms whose tokens mix the key channels, so that a chunk's effect on the state before it is a matrix.
+__host__ __device__ constexpr bool scan_mixes_keys(int mode) { return mode == SCAN_DELTA_RULE || mode == SCAN_GATED_DELTA; }
 __host__ __device__ constexpr int scan_tile(int mode) { return mode == SCAN_DELTA_RULE ? 16 : SCAN_TILE; }
 
 // SCAN_CHANNEL_DECAY: decay per key channel d = sigmoid(z[r, h, d])^(1 / p0), gain 1; the launcher turns the logits z
@@ -82,6 +92,10 @@ __host__ __device__ constexpr int scan_tile(int mode) { return mode == SCAN_DELT
 //                     launcher makes them from the projections before the scan.  A column first sums u . s over its key
 //                     channels (joined over the KS parts of a split column), then updates them.  In SCAN_LOCAL columns
 //                     Dv .. Dv + D - 1 carry the chunk's transition (see above) into ch.local_P.
+// SCAN_GATED_DELTA:   S~ = diag(a) S, S' = S~ + k (b (v - S~^T k))^T: per key channel a decay a (`gate` rows at g0), per head a
+//                     write strength b (`gate` rows at g1 + h).  The transition of a token is diag(a) - b k (k a)^T.
+// SCAN_HEAD_DECAY:    per head a decay (`gate` rows at g0 + h) and a gain (g1 + h): S' = decay S + gain k v^T.
+// Queries and keys may be shared by `qk_div` neighbouring heads: head h reads the columns of number h / qk_div.
 // PASS: SCAN_LOCAL / SCAN_FROM_START - launches (1) and (3) of the chunked form; grid z counts chunks.  Segments in one
 // piece are SCAN_FROM_START with chunks longer than any segment and no start states (`ch.start_S` null): from the slots.
 // grid (column blocks, heads, segments or chunks); a warp holds 32 / KS columns.  The exponential-gate form takes one
@@ -92,7 +106,7 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
     const float* __restrict__ proj, int P, int q_col, int k_col, int v_col, const float* __restrict__ gate, int gate_stride,
     int g0, int g1, float p0, float q_scale, float floor_, const int* __restrict__ seg_q_start,
     const int* __restrict__ seg_q_len, const int* __restrict__ seg_slot, float* __restrict__ memory,
-    float* __restrict__ normalizer, float* __restrict__ maximum, float* __restrict__ out, int H, int D, int Dv, ScanChunks ch) {
+    float* __restrict__ normalizer, float* __restrict__ maximum, float* __restrict__ out, int H, int D, int Dv, int qk_div, ScanChunks ch) {
     constexpr int RP = R + (KS > 1 ? 4 : 0);                   // a part's run in a staged row: 16 bytes of padding keep the parts' banks apart
     constexpr int RKP = RP * KS;                               // a staged row of key channels, zero beyond D
     constexpr int NPL = (R * KS + 31) / 32;                    // normaliser entries a lane keeps
@@ -102,7 +116,8 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
     const int part = lane % KS;                                // which run of R key channels of its column the lane holds
     const int VC = warps * COLS;                               // columns of the block
     const int col = blockIdx.x * VC + warp * COLS + lane / KS;
-    constexpr bool WITH_TRANSITION = MODE == SCAN_DELTA_RULE && PASS == SCAN_LOCAL;
+    constexpr bool WITH_TRANSITION = scan_mixes_keys(MODE) && PASS == SCAN_LOCAL;
+    constexpr bool CHANNEL_ROWS = MODE == SCAN_CHANNEL_DECAY || scan_mixes_keys(MODE);      // a row of decays is staged
     const bool col_ok = col < (WITH_TRANSITION ? Dv + D : Dv);
     int seg = blockIdx.z, chunk = 0, chunks = 1;
     if (!find_chunk(blockIdx.z, ch, seg_q_len, seg, chunk, chunks)) return;
@@ -121,7 +136,9 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
     extern __shared__ __align__(16) float tile_s[];
     constexpr int PARTS = scan_parts(MODE);
     constexpr int TILE = scan_tile(MODE);
-    const int tile_floats = TILE * (PARTS * RKP + VC);
+    constexpr int SCALARS = scan_scalars(MODE);
+    const int tile_floats = TILE * (PARTS * RKP + VC + SCALARS);
+    const int qk_off = h / qk_div * D;
     auto at = [](int d) { return (d / R) * RP + d % R; };      // where key channel d lies in a staged row
     auto stage = [&](int which, int first_row, int rows) {
         float* q_b = tile_s + (size_t)which * tile_floats;
@@ -132,9 +149,9 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
         for (int idx = threadIdx.x; idx < rows * D; idx += blockDim.x) {
             const int row = idx / D, d = idx - row * D;
             const float* src = proj + (size_t)(first_row + row) * P;
-            copy_async4(q_b + row * RKP + at(d), src + q_col + h * D + d);
-            copy_async4(k_b + row * RKP + at(d), src + k_col + h * D + d);
-            if (MODE != SCAN_EXP_GATES)
+            copy_async4(q_b + row * RKP + at(d), src + q_col + qk_off + d);
+            copy_async4(k_b + row * RKP + at(d), src + k_col + qk_off + d);
+            if (CHANNEL_ROWS)
                 copy_async4(a_b + row * RKP + at(d), gate + (size_t)(first_row + row) * gate_stride + g0 + h * D + d);
             if (MODE == SCAN_DELTA_RULE) {
                 const float* grow = gate + (size_t)(first_row + row) * gate_stride + g1 + h * D + d;
@@ -147,12 +164,22 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
             const int row = idx / v_cols, c = idx - row * v_cols;
             copy_async4(v_b + row * VC + c, proj + (size_t)(first_row + row) * P + v_col + h * Dv + blockIdx.x * VC + c);
         }
+        if (SCALARS > 0 && (int)threadIdx.x < rows) {           // a block has at least as many threads as a tile has tokens
+            float* s_b = v_b + TILE * VC;
+            const float* grow = gate + (size_t)(first_row + threadIdx.x) * gate_stride + h;
+            if (MODE == SCAN_HEAD_DECAY) {
+                copy_async4(s_b + threadIdx.x, grow + g0);
+                copy_async4(s_b + TILE + threadIdx.x, grow + g1);
+            } else {
+                copy_async4(s_b + threadIdx.x, grow + g1);
+            }
+        }
         copy_async_commit();
     };
     for (int idx = threadIdx.x; idx < 2 * tile_floats; idx += blockDim.x) tile_s[idx] = 0.f;
     __syncthreads();
     if (n_rows > 0) stage(0, r0, min(TILE, n_rows));
-    float S[R], nz[NPL], total[NPL];
+    float S[R], nz[NPL], total[NPL], total_keep = 1.f;
     float* mem = memory + ((size_t)slot * H + h) * D * Dv;
     const size_t cid = (size_t)blockIdx.z * H + h;             // (chunk id, head) in the scratch arrays
     const bool from_slot = ch.start_S == nullptr;
@@ -228,8 +255,13 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
         const float4* k4 = reinterpret_cast<const float4*>(k_s + tt * RKP + part * RP);
         const float4* a4 = reinterpret_cast<const float4*>(a_s + tt * RKP + part * RP);
         const float v = v_s[tt * VC + warp * COLS + lane / KS];
+        const float* s_s = v_s + TILE * VC + tt;               // the token's numbers per head
         float keep = 1.f, gain = v, denom = 1.f;
-        if (MODE == SCAN_EXP_GATES) {
+        if (MODE == SCAN_HEAD_DECAY) {
+            keep = s_s[0];
+            gain = s_s[TILE] * v;
+            if (PASS == SCAN_LOCAL) total_keep *= keep;
+        } else if (MODE == SCAN_EXP_GATES) {
             keep = gate_s[0][tt];
             const float take = gate_s[1][tt];
             gain = take * v;
@@ -243,7 +275,7 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
                 }
             }
             if (PASS != SCAN_LOCAL) denom = 1.f / (fmaxf(fabsf(warp_sum(dot) * q_scale), gate_s[2][tt]) + floor_);
-        } else if (PASS == SCAN_LOCAL && blockIdx.x == 0 && warp == 0) {
+        } else if (MODE == SCAN_CHANNEL_DECAY && PASS == SCAN_LOCAL && blockIdx.x == 0 && warp == 0) {
 #pragma unroll
             for (int i = 0; i < NPL; ++i) total[i] *= (lane + 32 * i < D) ? a_s[tt * RKP + at(lane + 32 * i)] : 1.f;
         }
@@ -267,13 +299,38 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
             read = -read;
             o0 = o1 = o2 = o3 = 0.f;
         }
+        if (MODE == SCAN_GATED_DELTA) {
+            // The column decays and is read along the key; what it is short of the value is written along the key below.
+#pragma unroll
+            for (int i = 0; i < R; i += 4) {
+                const float4 aa = a4[i >> 2], kk = k4[i >> 2];
+                S[i] *= aa.x;
+                S[i + 1] *= aa.y;
+                S[i + 2] *= aa.z;
+                S[i + 3] *= aa.w;
+                o0 = fmaf(kk.x, S[i], o0);
+                o1 = fmaf(kk.y, S[i + 1], o1);
+                o2 = fmaf(kk.z, S[i + 2], o2);
+                o3 = fmaf(kk.w, S[i + 3], o3);
+            }
+            read = (o0 + o1) + (o2 + o3);
+            if (KS >= 2) read += __shfl_xor_sync(0xffffffffu, read, 1);
+            if (KS == 4) read += __shfl_xor_sync(0xffffffffu, read, 2);
+            gain = s_s[0] * (v - read);
+            o0 = o1 = o2 = o3 = 0.f;
+        }
 #pragma unroll
         for (int i = 0; i < R; i += 4) {
             const float4 kk = k4[i >> 2];
             float4 qq = make_float4(0.f, 0.f, 0.f, 0.f), aa = make_float4(keep, keep, keep, keep);
             if (PASS != SCAN_LOCAL) qq = q4[i >> 2];
-            if (MODE != SCAN_EXP_GATES) aa = a4[i >> 2];
-            if (MODE == SCAN_DELTA_RULE) {
+            if (MODE == SCAN_CHANNEL_DECAY || MODE == SCAN_DELTA_RULE) aa = a4[i >> 2];
+            if (MODE == SCAN_GATED_DELTA) {
+                S[i] = fmaf(kk.x, gain, S[i]);
+                S[i + 1] = fmaf(kk.y, gain, S[i + 1]);
+                S[i + 2] = fmaf(kk.z, gain, S[i + 2]);
+                S[i + 3] = fmaf(kk.w, gain, S[i + 3]);
+            } else if (MODE == SCAN_DELTA_RULE) {
                 const float4 bb = b4[i >> 2];
                 S[i] = fmaf(aa.x, S[i], fmaf(bb.x, read, kk.x * gain));
                 S[i + 1] = fmaf(aa.y, S[i + 1], fmaf(bb.y, read, kk.y * gain));
@@ -314,6 +371,7 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
     }
     if (blockIdx.x != 0 || warp != 0) return;
     if (MODE != SCAN_EXP_GATES) {
+        if (PASS == SCAN_LOCAL && MODE == SCAN_HEAD_DECAY && lane == 0) ch.local_F[cid] = total_keep;
         if (PASS == SCAN_LOCAL && MODE == SCAN_CHANNEL_DECAY)
 #pragma unroll
             for (int i = 0; i < NPL; ++i) {
@@ -371,6 +429,8 @@ __global__ void scan_chunk_starts_kernel(const int* __restrict__ seg_q_len, cons
             if (c + 1 == chunks) break;
             if (MODE == SCAN_CHANNEL_DECAY) {
                 s = ch.local_vec[cid * D + d] * s + ch.local_S[cid * per + e];
+            } else if (MODE == SCAN_HEAD_DECAY) {
+                s = ch.local_F[cid] * s + ch.local_S[cid * per + e];
             } else {
                 const float F = ch.local_F[cid], ml = ch.local_m[cid];
                 const float m1 = fmaxf(F + m, ml);
@@ -396,7 +456,7 @@ __global__ void scan_chunk_starts_kernel(const int* __restrict__ seg_q_len, cons
         }
 }
 
-// Launch (2) for the delta rule: start[c + 1] = P[c] start[c] + local[c] - per chunk a product of the D x D transition with
+// Launch (2) for the delta rules: start[c + 1] = P[c] start[c] + local[c] - per chunk a product of the D x D transition with
 // the D x Dv state, the chunks in order.  A block holds 32 columns of the state of one (segment, head) and all key
 // channels; thread (ty, tx) of ceil(D / 4) x 8 holds rows 4 ty .. 4 ty + 3 and columns 4 tx .. 4 tx + 3 in registers.
 // The P[c] pass through a ring of shared-memory stages, 32 of their columns at a time and transposed (so that a thread's
@@ -506,15 +566,15 @@ __global__ void __launch_bounds__(512) delta_chunk_starts_kernel(const int* __re
 template <int MODE, int R, int KS>
 static int launch_scan(const float* proj, int P, int q_col, int k_col, int v_col, const float* gate, int gate_stride, int g0, int g1,
                         float p0, float q_scale, float floor_, const int* seg_q_start, const int* seg_q_len, const int* seg_slot,
-                        float* memory, float* normalizer, float* maximum, float* out, int S, int H, int D, int Dv, ScanChunks ch,
-                        int max_chunks, cudaStream_t stream) {
+                        float* memory, float* normalizer, float* maximum, float* out, int S, int H, int D, int Dv, int qk_div,
+                        ScanChunks ch, int max_chunks, cudaStream_t stream) {
     constexpr int COLS = 32 / KS;
     constexpr int RKP = (R + (KS > 1 ? 4 : 0)) * KS;
     const int total_warps = (Dv + COLS - 1) / COLS;
     // The exponential-gate form: all of a head's columns in one block (the caller chose KS so that they are at most 16
     // warps).  The other: blocks of up to 16 warps, fewer where the staging buffers would not fit.
     int warps = MODE == SCAN_EXP_GATES ? total_warps : (total_warps < 16 ? total_warps : 16);
-    auto bytes = [&](int w) { return 2 * (size_t)scan_tile(MODE) * (scan_parts(MODE) * RKP + w * COLS) * sizeof(float); };
+    auto bytes = [&](int w) { return 2 * (size_t)scan_tile(MODE) * (scan_parts(MODE) * RKP + w * COLS + scan_scalars(MODE)) * sizeof(float); };
     if (MODE != SCAN_EXP_GATES)
         while (warps > 1 && bytes(warps) > 200 * 1024) warps >>= 1;
     int col_blocks = (total_warps + warps - 1) / warps;
@@ -525,7 +585,7 @@ static int launch_scan(const float* proj, int P, int q_col, int k_col, int v_col
             cudaFuncSetAttribute(matrix_state_scan_kernel<MODE, R, KS, PASS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         kvb_launch(matrix_state_scan_kernel<MODE, R, KS, PASS>, dim3(col_blocks, H, Z), dim3(32 * warps), smem, stream, proj, P,    \
                    q_col, k_col, v_col, gate, gate_stride, g0, g1, p0, q_scale, floor_, seg_q_start, seg_q_len, seg_slot, memory,    \
-                   normalizer, maximum, out, H, D, Dv, ch);                                                                     \
+                   normalizer, maximum, out, H, D, Dv, qk_div, ch);                                                                     \
     } while (0)
     if (smem > 220 * 1024 || warps > 16) return KVB_ERR_LIMIT;
     if (max_chunks <= 0) {
@@ -536,7 +596,7 @@ static int launch_scan(const float* proj, int P, int q_col, int k_col, int v_col
         KVB_SCAN_PASS(SCAN_FROM_START, S);
         return KVB_OK;
     }
-    if constexpr (MODE == SCAN_DELTA_RULE) {
+    if constexpr (scan_mixes_keys(MODE)) {
         const int state_blocks = col_blocks;
         col_blocks = ((Dv + D + COLS - 1) / COLS + warps - 1) / warps;     // the transition's columns beside the state's
         KVB_SCAN_PASS(SCAN_LOCAL, max_chunks);
@@ -576,9 +636,12 @@ static int scan_any(int mode, const float* proj, int P, int q_col, int k_col, in
                     int gate_stride, int g0, int g1, float p0, float q_scale, float floor_, const int* seg_q_start,
                     const int* seg_q_len, const int* seg_slot, float* memory, float* normalizer, float* maximum,
                     float* out, int T, int S, int H, int D, int Dv, int chunk_len, int max_chunks, float* scratch,
-                    cudaStream_t stream, bool decays_ready = false) {
+                    cudaStream_t stream, bool decays_ready = false, int qk_heads = 0) {
     if (S <= 0) return KVB_OK;
-    if (H < 1 || D < 1 || Dv < 1 || mode < SCAN_CHANNEL_DECAY || mode > SCAN_DELTA_RULE) return KVB_ERR_SHAPE;
+    if (H < 1 || D < 1 || Dv < 1 || mode < SCAN_CHANNEL_DECAY || mode > SCAN_HEAD_DECAY) return KVB_ERR_SHAPE;
+    if (qk_heads <= 0) qk_heads = H;
+    if (H % qk_heads) return KVB_ERR_SHAPE;
+    const int qk_div = H / qk_heads;
     if (D > 256 || Dv > 512 || H > 65535 || S > 65535 || max_chunks > 65535) return KVB_ERR_LIMIT;
     if (max_chunks > 0 && (chunk_len < 1 || scratch == nullptr)) return KVB_ERR_SHAPE;
     ScanChunks ch = {};
@@ -607,7 +670,7 @@ static int scan_any(int mode, const float* proj, int P, int q_col, int k_col, in
     // lane took 312 us where 128 took 489 and 32 took 475; at 64 key channels one lane a column 129 us, four 160);
     // fewer lanes where the exponential-gate form's block (all of a head's columns) would pass 16 warps.
     int ks = D <= 64 ? 1 : D <= 128 ? 2 : 4;
-    if (mode == SCAN_DELTA_RULE && delta_rule_lanes > 0) ks = delta_rule_lanes;
+    if (scan_mixes_keys(mode) && delta_rule_lanes > 0) ks = delta_rule_lanes;
     if (mode == SCAN_EXP_GATES)
         while (ks > 1 && (Dv + 32 / ks - 1) / (32 / ks) > 16) ks >>= 1;
     const int per_lane = (D + ks - 1) / ks;
@@ -616,7 +679,7 @@ static int scan_any(int mode, const float* proj, int P, int q_col, int k_col, in
     int rc = KVB_ERR_LIMIT;
 #define KVB_SCAN(MODE, R, KS)                                                                                                  \
     rc = launch_scan<MODE, R, KS>(proj, P, q_col, k_col, v_col, gate, gate_stride, g0, g1, p0, q_scale, floor_, seg_q_start,   \
-                                  seg_q_len, seg_slot, memory, normalizer, maximum, out, S, H, D, Dv, ch, max_chunks, stream)
+                                  seg_q_len, seg_slot, memory, normalizer, maximum, out, S, H, D, Dv, qk_div, ch, max_chunks, stream)
 #define KVB_SCAN_KS(MODE, R)                                                                                                   \
     do {                                                                                                                      \
         if (ks == 4) KVB_SCAN(MODE, R, 4); else if (ks == 2) KVB_SCAN(MODE, R, 2); else KVB_SCAN(MODE, R, 1);                 \
@@ -628,6 +691,8 @@ static int scan_any(int mode, const float* proj, int P, int q_col, int k_col, in
     } while (0)
     if (mode == SCAN_CHANNEL_DECAY) KVB_SCAN_SIZE(SCAN_CHANNEL_DECAY);
     else if (mode == SCAN_EXP_GATES) KVB_SCAN_SIZE(SCAN_EXP_GATES);
+    else if (mode == SCAN_GATED_DELTA) KVB_SCAN_SIZE(SCAN_GATED_DELTA);
+    else if (mode == SCAN_HEAD_DECAY) KVB_SCAN_SIZE(SCAN_HEAD_DECAY);
     else KVB_SCAN_SIZE(SCAN_DELTA_RULE);
 #undef KVB_SCAN_SIZE
 #undef KVB_SCAN_KS
@@ -723,6 +788,244 @@ KVB_API int kvb_delta_rule_scan(const float* proj, int P, int r_col, int k_col, 
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Short causal convolutions.  A channel's output at a token is silu(bias + sum_n w[n] x(t - (taps - 1) + n)) over the inputs of
+// its own request, zero before the start; the last taps - 1 inputs of a request are its state, tail [slot, taps - 1, channel],
+// so that a portion finds them whatever way the request was cut.  Inputs are float32 columns col .. col + C of the rows `proj`,
+// weights [taps, C].
+struct ShortConv {
+    const float* proj;
+    int P, col, C, taps;
+    const float* w;
+    const float* bias;       // [C] or null
+    float* tail;             // [slots, taps - 1, C]
+    const int* row_segment;
+    const int* seg_q_start;
+    const int* seg_q_len;
+    const int* seg_slot;
+};
+
+struct ConvRow {             // where the inputs of one row lie
+    const float* row;        // the row's own inputs
+    float* tail;             // its request's state
+    int t;                   // how many rows of its segment come before it
+};
+
+__device__ __forceinline__ ConvRow conv_row(const ShortConv& cv, int r) {
+    const int seg = cv.row_segment[r];
+    return {cv.proj + (size_t)r * cv.P + cv.col, cv.tail + (size_t)cv.seg_slot[seg] * (cv.taps - 1) * cv.C, r - cv.seg_q_start[seg]};
+}
+
+// Channel c of the row.  `single`: every segment of the step is one row; the thread then also moves the channel's state on by
+// one token (it is the only one that touches it), otherwise short_conv_tail_kernel does so after this launch.
+__device__ __forceinline__ float conv_channel(const ShortConv& cv, const ConvRow& cr, int c, bool single) {
+    float acc = cv.bias ? cv.bias[c] : 0.f;
+    const float own = cr.row[c];
+    for (int n = 0; n + 1 < cv.taps; ++n) {
+        const int back = cv.taps - 1 - n;                      // this many tokens before the row
+        const float x = back <= cr.t ? cr.row[c - (long long)back * cv.P] : cr.tail[(size_t)(cv.taps - 1 - back + cr.t) * cv.C + c];
+        acc = fmaf(cv.w[(size_t)n * cv.C + c], x, acc);
+        if (single && n > 0) cr.tail[(size_t)(n - 1) * cv.C + c] = x;
+    }
+    if (single && cv.taps > 1) cr.tail[(size_t)(cv.taps - 2) * cv.C + c] = own;
+    acc = fmaf(cv.w[(size_t)(cv.taps - 1) * cv.C + c], own, acc);
+    return acc / (1.f + expf(-acc));
+}
+
+// The state after the step: a thread per (segment, channel).  Entry j moves from entry j + rows of the old state or from the
+// segment's rows; going up, an entry is read before it is overwritten.
+__global__ void short_conv_tail_kernel(ShortConv cv, int S) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seg = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= cv.C || seg >= S) return;
+    const int rows = cv.seg_q_len[seg];
+    const float* first = cv.proj + (size_t)cv.seg_q_start[seg] * cv.P + cv.col + c;
+    float* tail = cv.tail + (size_t)cv.seg_slot[seg] * (cv.taps - 1) * cv.C + c;
+    for (int j = 0; j < cv.taps - 1; ++j) {
+        const int at = rows - (cv.taps - 1) + j;
+        tail[(size_t)j * cv.C] = at >= 0 ? first[(size_t)at * cv.P] : tail[(size_t)(j + rows) * cv.C];
+    }
+}
+
+static int launch_conv_tail(const ShortConv& cv, int T, int S, cudaStream_t stream) {
+    if (T == S || cv.taps < 2) return KVB_OK;                  // single rows: the convolution has done it
+    kvb_launch(short_conv_tail_kernel, dim3((cv.C + 127) / 128, S), dim3(128), 0, stream, cv, S);
+    return kvb_launch_status();
+}
+
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+// What the gated delta rule reads, a warp per (row, job): the convolved, activated rows [q: G heads of D | k: G of D | v: H of Dv]
+// with q and k as unit vectors x / sqrt(sum x^2 + unit_eps) (jobs 0 .. 2 G - 1: a head each; then a head of v each), and
+// gates[r] = [decays a = exp(-rate_h softplus(z + dt_bias)): H of D | write strengths sigmoid(proj[b_col + h]): H] (a head each).
+__global__ void gated_delta_inputs_kernel(ShortConv cv, int b_col, const float* __restrict__ z, int z_stride, const float* __restrict__ dt_bias,
+                                          const float* __restrict__ rate, float unit_eps, float* __restrict__ rows,
+                                          float* __restrict__ gates, int total, int H, int G, int D, int Dv, int single) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (id >= total) return;
+    const int jobs = 2 * G + 2 * H, r = id / jobs, job = id - r * jobs;
+    float* out = rows + (size_t)r * cv.C;
+    if (job < 2 * G) {
+        const ConvRow cr = conv_row(cv, r);
+        float x[8], ss = 0.f;                                  // at most 256 channels a head
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int d = lane + 32 * i;
+            x[i] = d < D ? conv_channel(cv, cr, job * D + d, single) : 0.f;
+            ss += x[i] * x[i];
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) + unit_eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (lane + 32 * i < D) out[job * D + lane + 32 * i] = x[i] * inv;
+    } else if (job < 2 * G + H) {
+        const ConvRow cr = conv_row(cv, r);
+        const int c0 = 2 * G * D + (job - 2 * G) * Dv;
+        for (int d = lane; d < Dv; d += 32) out[c0 + d] = conv_channel(cv, cr, c0 + d, single);
+    } else {
+        const int h = job - 2 * G - H;
+        float* g = gates + (size_t)r * (H * D + H);
+        const float* zr = z + (size_t)r * z_stride + h * D;
+        const float rt = rate[h];
+        for (int d = lane; d < D; d += 32) g[h * D + d] = expf(-rt * softplus(zr[d] + dt_bias[h * D + d]));
+        if (lane == 0) g[H * D + h] = 1.f / (1.f + expf(-cv.proj[(size_t)r * cv.P + b_col + h]));
+    }
+}
+
+// proj: float32 [T, P] with the projections [q | k | v] at `col` and the write-strength logits at `b_col`; z: the decay logits
+// (columns 0 .. H * D of rows of z_stride); rate [H] = exp of the learned log rates; rows [T, 2 G D + H Dv] and gates
+// [T, H D + H] float32 are what kvb_gated_delta_scan reads.  `tail` moves on by the step's rows.
+KVB_API int kvb_gated_delta_inputs(const float* proj, int P, int col, int b_col, const float* conv_w, int taps, float* tail, const float* z,
+                                   int z_stride, const float* dt_bias, const float* rate, float unit_eps, float* rows, float* gates,
+                                   const int* row_segment, const int* seg_q_start, const int* seg_q_len, const int* seg_slot, int T, int S,
+                                   int H, int G, int D, int Dv, cudaStream_t stream) {
+    if (T <= 0 || S <= 0) return KVB_OK;
+    if (H < 1 || G < 1 || H % G || D < 1 || Dv < 1 || taps < 1 || z_stride < H * D) return KVB_ERR_SHAPE;
+    if (D > 256 || S > 65535 || (long long)T * (2 * G + 2 * H) > 0x7fffffffLL) return KVB_ERR_LIMIT;
+    const ShortConv cv = {proj, P, col, 2 * G * D + H * Dv, taps, conv_w, nullptr, tail, row_segment, seg_q_start, seg_q_len, seg_slot};
+    const int total = T * (2 * G + 2 * H), warps = 4;
+    kvb_launch(gated_delta_inputs_kernel, dim3((total + warps - 1) / warps), dim3(32 * warps), 0, stream, cv, b_col, z, z_stride, dt_bias,
+               rate, unit_eps, rows, gates, total, H, G, D, Dv, T == S ? 1 : 0);
+    return launch_conv_tail(cv, T, S, stream);
+}
+
+// The gated delta rule over the tokens of every segment, from and into memory[slot] ([H, D, Dv], float32); rows and gates as made
+// by kvb_gated_delta_inputs.  out = q_scale S'^T q.  `max_chunks` > 0: the chunked form, as for the other scans, with `scratch`
+// of max_chunks * H * (2 D Dv + D D + 2 D + 3) floats.
+KVB_API int kvb_gated_delta_scan(const float* rows, const float* gates, float q_scale, const int* seg_q_start, const int* seg_q_len,
+                                 const int* seg_slot, float* memory, float* out, int T, int S, int H, int G, int D, int Dv, int chunk_len,
+                                 int max_chunks, float* scratch, cudaStream_t stream) {
+    if (S <= 0 || T <= 0) return KVB_OK;
+    if (G < 1 || H % G) return KVB_ERR_SHAPE;
+    return scan_any(SCAN_GATED_DELTA, rows, 2 * G * D + H * Dv, 0, G * D, 2 * G * D, gates, H * D + H, 0, H * D, 0.f, q_scale, 0.f, seg_q_start,
+                    seg_q_len, seg_slot, memory, nullptr, nullptr, out, T, S, H, D, Dv, chunk_len, max_chunks, scratch, stream, true, G);
+}
+
+// What the state-space recurrence reads, a warp per (row, job): a run of 128 convolved, activated channels each, then (the last
+// job) gates[r] = [exp(-rate_h d_h): H | d_h: H] with d = softplus(proj[dt_col + h] + dt_bias_h).
+constexpr int CONV_RUN = 128;
+__global__ void state_space_inputs_kernel(ShortConv cv, int dt_col, const float* __restrict__ dt_bias, const float* __restrict__ rate,
+                                          float* __restrict__ rows, float* __restrict__ gates, int total, int H, int single) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (id >= total) return;
+    const int jobs = (cv.C + CONV_RUN - 1) / CONV_RUN + 1, r = id / jobs, job = id - r * jobs;
+    if (job + 1 < jobs) {
+        const ConvRow cr = conv_row(cv, r);
+        float* out = rows + (size_t)r * cv.C;
+        const int end = min(cv.C, (job + 1) * CONV_RUN);
+        for (int c = job * CONV_RUN + lane; c < end; c += 32) out[c] = conv_channel(cv, cr, c, single);
+    } else {
+        float* g = gates + (size_t)r * 2 * H;
+        for (int h = lane; h < H; h += 32) {
+            const float d = softplus(cv.proj[(size_t)r * cv.P + dt_col + h] + dt_bias[h]);
+            g[h] = expf(-rate[h] * d);
+            g[H + h] = d;
+        }
+    }
+}
+
+// proj: float32 [T, P] with the C convolved channels [x: H Dv | B: G N | C: G N] at `col` and the step sizes at `dt_col`; rows
+// [T, C] and gates [T, 2 H] float32 are what kvb_state_space_scan reads.  `tail` moves on by the step's rows.
+KVB_API int kvb_state_space_inputs(const float* proj, int P, int col, int C, int dt_col, const float* conv_w, const float* conv_b, int taps,
+                                   float* tail, const float* dt_bias, const float* rate, float* rows, float* gates, const int* row_segment,
+                                   const int* seg_q_start, const int* seg_q_len, const int* seg_slot, int T, int S, int H,
+                                   cudaStream_t stream) {
+    if (T <= 0 || S <= 0) return KVB_OK;
+    if (H < 1 || C < 1 || taps < 1) return KVB_ERR_SHAPE;
+    const int jobs = (C + CONV_RUN - 1) / CONV_RUN + 1, warps = 4;
+    if (S > 65535 || (long long)T * jobs > 0x7fffffffLL) return KVB_ERR_LIMIT;
+    const ShortConv cv = {proj, P, col, C, taps, conv_w, conv_b, tail, row_segment, seg_q_start, seg_q_len, seg_slot};
+    const int total = T * jobs;
+    kvb_launch(state_space_inputs_kernel, dim3((total + warps - 1) / warps), dim3(32 * warps), 0, stream, cv, dt_col, dt_bias, rate, rows,
+               gates, total, H, T == S ? 1 : 0);
+    return launch_conv_tail(cv, T, S, stream);
+}
+
+// S' = decay S + d B x^T, out = S'^T C over the tokens of every segment, from and into memory[slot] ([H, N, Dv], float32); head h
+// reads B and C of group h / (H / G); rows and gates as made by kvb_state_space_inputs.
+KVB_API int kvb_state_space_scan(const float* rows, const float* gates, const int* seg_q_start, const int* seg_q_len, const int* seg_slot,
+                                 float* memory, float* out, int T, int S, int H, int G, int N, int Dv, int chunk_len, int max_chunks,
+                                 float* scratch, cudaStream_t stream) {
+    if (S <= 0 || T <= 0) return KVB_OK;
+    if (G < 1 || H % G) return KVB_ERR_SHAPE;
+    return scan_any(SCAN_HEAD_DECAY, rows, H * Dv + 2 * G * N, H * Dv + G * N, H * Dv, 0, gates, 2 * H, 0, H, 0.f, 1.f, 0.f, seg_q_start,
+                    seg_q_len, seg_slot, memory, nullptr, nullptr, out, T, S, H, N, Dv, chunk_len, max_chunks, scratch, stream, true, G);
+}
+
+// out[t, out_col + i] = y_i / sqrt(mean over i's part of y^2 + eps) * w_i * scale with y_i = (o[t, i] + skip[i / Dv] x[t, i]) silu(g[t, i]);
+// a row's W = H Dv numbers form `parts` equal parts, a block each.  o, x, g float32 (x and g columns of wider rows).
+template <typename T>
+__global__ void gate_part_norm_kernel(const float* __restrict__ o, const float* __restrict__ x, int x_stride, const float* __restrict__ skip,
+                                      const float* __restrict__ gate, int gate_stride, int gate_col, const float* __restrict__ w, float eps,
+                                      float scale, T* __restrict__ out, int out_stride, int out_col, int W, int Dv, int n) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float scratch[33];
+    extern __shared__ float y_s[];
+    const int t = blockIdx.x, i0 = blockIdx.y * n;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const int c = i0 + i;
+        const float z = gate[(size_t)t * gate_stride + gate_col + c];
+        const float y = fmaf(skip[c / Dv], x[(size_t)t * x_stride + c], o[(size_t)t * W + c]) * (z / (1.f + expf(-z)));
+        y_s[i] = y;
+        ss += y * y;
+    }
+    const float inv = scale / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+    for (int i = threadIdx.x; i < n; i += blockDim.x)
+        out[(size_t)t * out_stride + out_col + i0 + i] = from_f32<T>(y_s[i] * inv * w[i0 + i]);
+}
+
+KVB_API int kvb_gate_part_norm(int out_dtype, const float* o, const float* x, int x_stride, const float* skip, const float* gate, int gate_stride,
+                               int gate_col, const float* w, float eps, float scale, void* out, int out_stride, int out_col, int T, int H, int Dv,
+                               int parts, cudaStream_t stream) {
+    if (T <= 0) return KVB_OK;
+    const int W = H * Dv;
+    if (H < 1 || Dv < 1 || parts < 1 || W % parts) return KVB_ERR_SHAPE;
+    const int n = W / parts, threads = n >= 2048 ? 512 : n >= 512 ? 256 : n >= 128 ? 128 : 64;
+    const size_t smem = (size_t)n * sizeof(float);
+    if (parts > 65535 || smem > 200 * 1024) return KVB_ERR_LIMIT;
+    if (out_dtype == KVB_F32) {
+        if (smem > 46 * 1024) cudaFuncSetAttribute(gate_part_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        kvb_launch(gate_part_norm_kernel<float>, dim3(T, parts), dim3(threads), smem, stream, o, x, x_stride, skip, gate, gate_stride, gate_col,
+                   w, eps, scale, (float*)out, out_stride, out_col, W, Dv, n);
+    } else if (out_dtype == KVB_BF16) {
+        if (smem > 46 * 1024) cudaFuncSetAttribute(gate_part_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        kvb_launch(gate_part_norm_kernel<bf16>, dim3(T, parts), dim3(threads), smem, stream, o, x, x_stride, skip, gate, gate_stride, gate_col,
+                   w, eps, scale, (bf16*)out, out_stride, out_col, W, Dv, n);
+    } else {
+        return KVB_ERR_DTYPE;
+    }
+    return kvb_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // One warp per (row, head).  o: float32 [T, H * Dv]; w: [Dv] (shared by the heads) or [H * Dv] (w_per_head);
 // gate: float32 rows of stride gate_stride, the head's Dv numbers at gate_col + h * Dv; act 0: silu, 1: sigmoid.
 // out (type T) rows of stride out_stride, written at out_col + h * Dv.
@@ -803,40 +1106,70 @@ KVB_API int kvb_head_norm_gate(int out_dtype, const float* o, const float* w, in
     return kvb_launch_status();
 }
 
-// out[t, out_col + h * Dv + d] = x[t, h * xs + d] * sigmoid(gate[t, gate_col + h]) * scale (gate null: no sigmoid); xs >= Dv:
-// a head of x may carry columns after its Dv numbers, which are left out.
-template <typename T>
-__global__ void head_gate_kernel(const T* __restrict__ x, int xs, const T* __restrict__ gate, int gate_stride, int gate_col, float scale,
-                                 T* __restrict__ out, int out_stride, int out_col, int H, int Dv, size_t total) {
+// out[t, out_col + h * Dv + d] = x[t, h * xs + d] * sigmoid(g) * scale, g = gate[t, gate_col + h], or with `per_channel`
+// gate[t, gate_col + h * Dv + d] (gate null: no sigmoid); xs >= Dv: a head of x may carry columns after its Dv numbers, which
+// are left out.  A thread takes VEC neighbouring numbers of one head (all of x, gate, out then start on a VEC boundary).
+template <typename T, int VEC>
+__global__ void head_gate_kernel(const T* __restrict__ x, int xs, const T* __restrict__ gate, int gate_stride, int gate_col, int per_channel,
+                                 float scale, T* __restrict__ out, int out_stride, int out_col, int H, int Dv, int total) {
     pdl_wait();
     pdl_launch_dependents();
-    const int width = H * Dv;
-    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = idx / width;
-        const int c = (int)(idx - t * width);
-        float v = to_f32<T>(x[(t * H + c / Dv) * xs + c % Dv]) * scale;
-        if (gate) v *= 1.f / (1.f + expf(-to_f32<T>(gate[t * gate_stride + gate_col + c / Dv])));
-        out[t * out_stride + out_col + c] = from_f32<T>(v);
+    struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
+    const int per_row = H * Dv / VEC;
+    for (int idx = blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += gridDim.x * blockDim.x) {
+        const int t = idx / per_row, c = (idx - t * per_row) * VEC, h = c / Dv, d = c - h * Dv;
+        const Pack in = *reinterpret_cast<const Pack*>(x + ((size_t)t * H + h) * xs + d);
+        float s[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s[e] = scale;
+        if (gate && per_channel) {
+            const Pack g = *reinterpret_cast<const Pack*>(gate + (size_t)t * gate_stride + gate_col + c);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) s[e] = scale / (1.f + expf(-to_f32<T>(g.v[e])));
+        } else if (gate) {
+            const float one = scale / (1.f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + gate_col + h])));
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) s[e] = one;
+        }
+        Pack o;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) o.v[e] = from_f32<T>(to_f32<T>(in.v[e]) * s[e]);
+        *reinterpret_cast<Pack*>(out + (size_t)t * out_stride + out_col + c) = o;
     }
 }
 
-KVB_API int kvb_head_gate(int dtype, const void* x, int xs, const void* gate, int gate_stride, int gate_col, float scale, void* out,
-                          int out_stride, int out_col, int T, int H, int Dv, cudaStream_t stream) {
-    const size_t total = (size_t)T * H * Dv;
-    if (total == 0) return KVB_OK;
-    if (xs < Dv) return KVB_ERR_SHAPE;
-    size_t blocks = (total + 255) / 256;
-    const size_t most = (size_t)kvb_sm_count() * 16;
+template <typename T>
+static int launch_head_gate(const T* x, int xs, const T* gate, int gate_stride, int gate_col, int per_channel, float scale, T* out,
+                            int out_stride, int out_col, int T_, int H, int Dv, cudaStream_t stream) {
+    constexpr int V = 16 / (int)sizeof(T);
+    const bool wide = Dv % V == 0 && xs % V == 0 && out_stride % V == 0 && out_col % V == 0 &&
+                      (!(gate && per_channel) || (gate_stride % V == 0 && gate_col % V == 0)) &&
+                      ((((uintptr_t)x) | ((uintptr_t)out) | (gate && per_channel ? (uintptr_t)gate : 0)) & 15) == 0;
+    const long long total = (long long)T_ * H * Dv / (wide ? V : 1);
+    if (total > 0x7fffffffLL - (1 << 24)) return KVB_ERR_LIMIT;
+    long long blocks = (total + 127) / 128;
+    const long long most = (long long)kvb_sm_count() * 32;
     if (blocks > most) blocks = most;
-    if (dtype == KVB_F32)
-        kvb_launch(head_gate_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, (const float*)x, xs, (const float*)gate, gate_stride,
-                   gate_col, scale, (float*)out, out_stride, out_col, H, Dv, total);
-    else if (dtype == KVB_BF16)
-        kvb_launch(head_gate_kernel<bf16>, dim3((int)blocks), dim3(256), 0, stream, (const bf16*)x, xs, (const bf16*)gate, gate_stride,
-                   gate_col, scale, (bf16*)out, out_stride, out_col, H, Dv, total);
+    if (wide)
+        kvb_launch(head_gate_kernel<T, V>, dim3((unsigned)blocks), dim3(128), 0, stream, x, xs, gate, gate_stride, gate_col, per_channel, scale,
+                   out, out_stride, out_col, H, Dv, (int)total);
     else
-        return KVB_ERR_DTYPE;
+        kvb_launch(head_gate_kernel<T, 1>, dim3((unsigned)blocks), dim3(128), 0, stream, x, xs, gate, gate_stride, gate_col, per_channel, scale,
+                   out, out_stride, out_col, H, Dv, (int)total);
     return kvb_launch_status();
+}
+
+KVB_API int kvb_head_gate(int dtype, const void* x, int xs, const void* gate, int gate_stride, int gate_col, int per_channel, float scale,
+                          void* out, int out_stride, int out_col, int T, int H, int Dv, cudaStream_t stream) {
+    if (T <= 0 || H <= 0 || Dv <= 0) return KVB_OK;
+    if (xs < Dv) return KVB_ERR_SHAPE;
+    if (dtype == KVB_F32)
+        return launch_head_gate<float>((const float*)x, xs, (const float*)gate, gate_stride, gate_col, per_channel, scale, (float*)out,
+                                       out_stride, out_col, T, H, Dv, stream);
+    if (dtype == KVB_BF16)
+        return launch_head_gate<bf16>((const bf16*)x, xs, (const bf16*)gate, gate_stride, gate_col, per_channel, scale, (bf16*)out, out_stride,
+                                      out_col, T, H, Dv, stream);
+    return KVB_ERR_DTYPE;
 }
 
 // ---------------------------------------------------------------------------------------------------------------

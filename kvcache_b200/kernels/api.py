@@ -91,7 +91,7 @@ _SIGNATURES = {
                       _c_void_p],
         "kvb_token_shift": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                             _c_int, _c_int, _c_void_p],
-        "kvb_activation": [_c_int, _c_void_p, _c_longlong, _c_int, _c_float, _c_void_p],
+        "kvb_activation": [_c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_longlong, _c_int, _c_int, _c_float, _c_void_p],
         "kvb_add_norm": [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float,
                          _c_void_p],
         "kvb_silu_mul": [_c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
@@ -116,8 +116,19 @@ _SIGNATURES = {
         "kvb_delta_rule_set_lanes": [_c_int],
         "kvb_head_norm_gate": [_c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p,
                                _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
-        "kvb_head_gate": [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                          _c_void_p],
+        "kvb_head_gate": [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_int,
+                          _c_int, _c_void_p],
+        "kvb_gated_delta_inputs": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
+                                   _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
+                                   _c_int, _c_int, _c_int, _c_void_p],
+        "kvb_gated_delta_scan": [_c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+        "kvb_state_space_inputs": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
+                                   _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
+        "kvb_state_space_scan": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
+                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+        "kvb_gate_part_norm": [_c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_float, _c_float,
+                               _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_lightning_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                                _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
         "kvb_bigram_embed": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
@@ -464,15 +475,21 @@ class CudaKernels(KernelSet):
                                                  _ptr(batch.row_segment), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len),
                                                  _ptr(batch.seg_slot), _ptr(out), T, H, self._stream()), "token_shift")
 
-    ACTIVATIONS = {"tanh": 0, "relu2": 1, "softcap": 2}
+    ACTIVATIONS = {"tanh": 0, "relu2": 1, "softcap": 2, "gelu": 3}
 
     def activation_(self, x: torch.Tensor, kind: str, cap: float = 0.0) -> None:
-        """x = tanh(x), relu(x)^2 or cap * tanh(x / cap) ("softcap"), in place."""
+        """x = tanh(x), relu(x)^2, cap * tanh(x / cap) ("softcap") or x Phi(x) ("gelu", the exact one), in place."""
+        self.activation_into(x, kind, x, cap=cap)
+
+    def activation_into(self, x: torch.Tensor, kind: str, out: torch.Tensor, out_col: int = 0, cap: float = 0.0) -> None:
+        """out[:, out_col : out_col + x.shape[1]] = act(x), see `activation_`."""
         if kind not in self.ACTIVATIONS:
-            raise KernelError(f"activation_: '{kind}' is not built")
+            raise KernelError(f"activation_into: '{kind}' is not built")
+        if x.dtype != out.dtype or x.shape[0] != out.shape[0]:
+            raise KernelError("activation_into: rows of one type, as many on either side")
         self._count("activation")
-        _check(self._elementwise.kvb_activation(_dtype_code(x.dtype), _ptr(x), x.numel(), self.ACTIVATIONS[kind], float(cap),
-                                                self._stream()), "activation")
+        _check(self._elementwise.kvb_activation(_dtype_code(x.dtype), _ptr(x), x.shape[1], 0, _ptr(out), out.shape[1], out_col, x.shape[0],
+                                                x.shape[1], self.ACTIVATIONS[kind], float(cap), self._stream()), "activation")
 
     # ---- the folded chain of a decode layer ------------------------------------------------------------------
     # For steps of few rows a layer can run as five launches instead of eight: the norm before a product inside that
@@ -1213,8 +1230,9 @@ class CudaKernels(KernelSet):
             self._stream()), "bigram_embed")
 
     def head_gate(self, x: torch.Tensor, gate, num_heads: int, value_dim: int, scale: float, out: torch.Tensor,
-                  out_col: int = 0, x_head_stride: Optional[int] = None) -> None:
+                  out_col: int = 0, x_head_stride: Optional[int] = None, per_channel: bool = False) -> None:
         """out[t, out_col + h * Dv + d] = x[t, h * xs + d] * sigmoid(g[t, col + h]) * scale; `gate` = (g, col) or None;
+        `per_channel`: a gate for every number, g[t, col + h * Dv + d];
         xs = `x_head_stride` (None: Dv): a head of x may carry columns after its Dv numbers, which are left out."""
         T = x.shape[0]
         xs = value_dim if x_head_stride is None else int(x_head_stride)
@@ -1224,8 +1242,8 @@ class CudaKernels(KernelSet):
         if g is not None and g.dtype != x.dtype:
             raise KernelError("head_gate: the gate and the rows differ in type")
         self._count("head_gate")
-        _check(self._recurrent.kvb_head_gate(_dtype_code(x.dtype), _ptr(x), xs, _ptr(g), 0 if g is None else g.shape[1], col, float(scale),
-                                             _ptr(out), out.shape[1], out_col, T, num_heads, value_dim, self._stream()), "head_gate")
+        _check(self._recurrent.kvb_head_gate(_dtype_code(x.dtype), _ptr(x), xs, _ptr(g), 0 if g is None else g.shape[1], col,
+                                             1 if per_channel else 0, float(scale), _ptr(out), out.shape[1], out_col, T, num_heads, value_dim, self._stream()), "head_gate")
 
     def head_norm_gate(self, o: torch.Tensor, weight: torch.Tensor, eps: float, gate, activation: str, scale: float,
                        out: torch.Tensor, out_col: int, num_heads: int, value_dim: int, scope: str = "head") -> None:
@@ -1340,6 +1358,99 @@ class CudaKernels(KernelSet):
             _ptr(proj), proj.shape[1], cols[0], cols[1], cols[2], cols[3], _ptr(z), float(rate), float(unit_eps), _ptr(aux),
             _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out), T, batch.num_segments,
             H, D, chunk, max_chunks, _ptr(scratch), self._stream()), "delta_rule_scan")
+
+    def _chunks(self, batch: StepBatch, workspace, floats_per_chunk: int, chunk: int):
+        """(chunk bound, scratch) of a scan in chunks of `chunk` tokens, or (0, None) where segments are scanned in one piece.
+        Sized by the step's rows and segments alone, so that a recorded step finds the same launches."""
+        if not self.SCAN_CHUNK or batch.max_q_len < self.SCAN_CHUNK_MIN_ROWS:
+            return 0, None
+        self.launches += 2
+        bound = -(-batch.num_tokens // chunk) + batch.num_segments
+        return bound, workspace.buffer("recurrent.mixing_chunks", (bound * floats_per_chunk,), torch.float32)
+
+    def _conv_launches(self, batch: StepBatch, taps: int) -> None:
+        self.launches += 1 if batch.num_tokens != batch.num_segments and taps > 1 else 0     # the state's own launch
+
+    @staticmethod
+    def _float32_only(what: str, *tensors: torch.Tensor) -> None:
+        if any(t is not None and t.dtype != torch.float32 for t in tensors):
+            raise KernelError(f"{what} takes float32 rows, weights and states")
+
+    def gated_delta_inputs(self, proj: torch.Tensor, b_col: int, conv_w: torch.Tensor, tail: torch.Tensor, z: torch.Tensor,
+                           dt_bias: torch.Tensor, rate: torch.Tensor, unit_eps: float, batch: StepBatch, rows: torch.Tensor,
+                           gates: torch.Tensor, H: int, G: int, D: int, Dv: int) -> None:
+        """rows = silu of the causal convolution (weights `conv_w` [taps, channels]) of columns [q: G D | k: G D | v: H Dv] of
+        `proj`, q and k divided by sqrt(sum of squares + unit_eps) per head; gates = [exp(-rate_h softplus(z + dt_bias)): H D |
+        sigmoid(proj[:, b_col + h]): H].  `tail` [slots, taps - 1, channels]: the request's last inputs, moved on."""
+        self._float32_only("gated_delta_inputs", proj, conv_w, tail, z, dt_bias, rate, rows, gates)
+        T, C, taps = proj.shape[0], 2 * G * D + H * Dv, conv_w.shape[0]
+        if (tuple(conv_w.shape) != (taps, C) or tuple(tail.shape[1:]) != (taps - 1, C) or tuple(rows.shape) != (T, C)
+                or tuple(gates.shape) != (T, H * D + H) or dt_bias.numel() != H * D or rate.numel() != H or b_col < C):
+            raise KernelError("gated_delta_inputs: the sizes do not fit one another")
+        self._count("gated_delta_inputs")
+        self._conv_launches(batch, taps)
+        _check(self._recurrent.kvb_gated_delta_inputs(
+            _ptr(proj), proj.shape[1], 0, b_col, _ptr(conv_w), taps, _ptr(tail), _ptr(z), z.shape[1], _ptr(dt_bias), _ptr(rate),
+            float(unit_eps), _ptr(rows), _ptr(gates), _ptr(batch.row_segment), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len),
+            _ptr(batch.seg_slot), T, batch.num_segments, H, G, D, Dv, self._stream()), "gated_delta_inputs")
+
+    def gated_delta_scan(self, rows: torch.Tensor, gates: torch.Tensor, q_scale: float, batch: StepBatch, memory: torch.Tensor,
+                         out: torch.Tensor, H: int, G: int, D: int, Dv: int, workspace) -> None:
+        """Per segment, from and into memory[slot] ([H, D, Dv], float32): S~ = diag(a) S, S = S~ + k (b (v - S~^T k))^T,
+        out = q_scale S^T q; `rows` and `gates` as `gated_delta_inputs` makes them (head h: query and key h // (H / G))."""
+        self._float32_only("gated_delta_scan", rows, gates, memory, out)
+        if tuple(memory.shape[1:]) != (H, D, Dv):
+            raise KernelError(f"the gated delta scan wants states [slots, {H}, {D}, {Dv}], got {tuple(memory.shape)}")
+        chunk = self.SCAN_CHUNK if batch.max_q_len < self.DELTA_LONG_ROWS else max(self.SCAN_CHUNK, self.DELTA_LONG_CHUNK)
+        max_chunks, scratch = self._chunks(batch, workspace, H * (2 * D * Dv + D * D + 2 * D + 3), chunk)
+        self._count("gated_delta_scan")
+        _check(self._recurrent.kvb_gated_delta_scan(
+            _ptr(rows), _ptr(gates), float(q_scale), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory),
+            _ptr(out), rows.shape[0], batch.num_segments, H, G, D, Dv, chunk, max_chunks, _ptr(scratch), self._stream()), "gated_delta_scan")
+
+    def state_space_inputs(self, proj: torch.Tensor, col: int, dt_col: int, conv_w: torch.Tensor, conv_b: torch.Tensor, tail: torch.Tensor,
+                           dt_bias: torch.Tensor, rate: torch.Tensor, batch: StepBatch, rows: torch.Tensor, gates: torch.Tensor,
+                           H: int) -> None:
+        """rows = silu of the causal convolution (weights [taps, C], bias [C]) of columns col .. col + C of `proj`;
+        gates = [exp(-rate_h d_h): H | d_h: H], d = softplus(proj[:, dt_col + h] + dt_bias_h).  `tail` as above."""
+        self._float32_only("state_space_inputs", proj, conv_w, conv_b, tail, dt_bias, rate, rows, gates)
+        T, (taps, C) = proj.shape[0], conv_w.shape
+        if (conv_b.numel() != C or tuple(tail.shape[1:]) != (taps - 1, C) or tuple(rows.shape) != (T, C) or tuple(gates.shape) != (T, 2 * H)
+                or dt_bias.numel() != H or rate.numel() != H or max(col + C, dt_col + H) > proj.shape[1]):
+            raise KernelError("state_space_inputs: the sizes do not fit one another")
+        self._count("state_space_inputs")
+        self._conv_launches(batch, taps)
+        _check(self._recurrent.kvb_state_space_inputs(
+            _ptr(proj), proj.shape[1], col, C, dt_col, _ptr(conv_w), _ptr(conv_b), taps, _ptr(tail), _ptr(dt_bias), _ptr(rate), _ptr(rows),
+            _ptr(gates), _ptr(batch.row_segment), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), T,
+            batch.num_segments, H, self._stream()), "state_space_inputs")
+
+    def state_space_scan(self, rows: torch.Tensor, gates: torch.Tensor, batch: StepBatch, memory: torch.Tensor, out: torch.Tensor, H: int,
+                         G: int, N: int, Dv: int, workspace) -> None:
+        """Per segment, from and into memory[slot] ([H, N, Dv], float32): S = decay S + d B x^T, out = S^T C; `rows` =
+        [x: H Dv | B: G N | C: G N] and `gates` = [decay: H | d: H] as `state_space_inputs` makes them (head h: group h // (H / G))."""
+        self._float32_only("state_space_scan", rows, gates, memory, out)
+        if tuple(memory.shape[1:]) != (H, N, Dv) or rows.shape[1] != H * Dv + 2 * G * N:
+            raise KernelError(f"the state-space scan wants states [slots, {H}, {N}, {Dv}], got {tuple(memory.shape)}")
+        max_chunks, scratch = self._chunks(batch, workspace, H * (2 * N * Dv + 2 * N + 3), self.SCAN_CHUNK)
+        self._count("state_space_scan")
+        _check(self._recurrent.kvb_state_space_scan(
+            _ptr(rows), _ptr(gates), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out),
+            rows.shape[0], batch.num_segments, H, G, N, Dv, self.SCAN_CHUNK, max_chunks, _ptr(scratch), self._stream()), "state_space_scan")
+
+    def gate_part_norm(self, o: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, gate, weight: torch.Tensor, eps: float, scale: float,
+                       out: torch.Tensor, out_col: int, num_heads: int, value_dim: int, parts: int) -> None:
+        """y = (o + skip_h x) silu(g), a row's num_heads * value_dim numbers in `parts` equal parts; out[:, out_col + i] =
+        y_i / sqrt(mean of y^2 over i's part + eps) * weight_i * scale.  `x`: columns 0 .. of wider rows; `gate` = (g, col)."""
+        g, col = gate
+        self._float32_only("gate_part_norm", o, x, skip, g, weight)
+        W = num_heads * value_dim
+        if o.shape[1] != W or weight.numel() != W or skip.numel() != num_heads or W % parts:
+            raise KernelError("gate_part_norm: the sizes do not fit one another")
+        self._count("gate_part_norm")
+        _check(self._recurrent.kvb_gate_part_norm(
+            _dtype_code(out.dtype), _ptr(o), _ptr(x), x.shape[1], _ptr(skip), _ptr(g), g.shape[1], col, _ptr(weight), float(eps), float(scale),
+            _ptr(out), out.shape[1], out_col, o.shape[0], num_heads, value_dim, parts, self._stream()), "gate_part_norm")
 
     def sample(self, logits: torch.Tensor, temperature: torch.Tensor, seeds: torch.Tensor, counters: torch.Tensor,
                out: torch.Tensor, scratch_val: torch.Tensor, scratch_idx: torch.Tensor) -> None:

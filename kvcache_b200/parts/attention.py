@@ -37,6 +37,9 @@ class GQAAttention(Mixer):
     tensor-core kernels, which take one size for both (bfloat16, keys of up to 128 numbers in steps of 16); the heads'
     results then carry those zero columns, which the step after attention leaves out.
 
+    `head_gate_scope` "channel": the gate is one number per number of the heads' results instead of one per head (`head_gate`
+    then names a [heads * value_dim, hidden] matrix).
+
     `chunk`: a query sees the keys of its own chunk of this many tokens, counted from the request's first, up to itself (not
     beside a window).  `rotary_layout` "interleaved": the rotation pairs neighbours (2 t, 2 t + 1) instead of dimensions half
     the rotated ones apart; the rows of the projections are reordered when they are bound.  `out_bias`: the output matrix has
@@ -52,7 +55,8 @@ class GQAAttention(Mixer):
                  qk_norm_scope: str = "head", qk_norm_weight: bool = True, qk_norm_after_rotation: bool = False,
                  sink=None, keep_first: int = 0, value_mix: Optional[str] = None, value_mix_name: str = "vmix",
                  q_temperature=None, score_cap: Optional[float] = None, distance_bias: Optional[str] = None,
-                 pad_values: bool = False, chunk: Optional[int] = None, rotary_layout: str = "half", own_kv: bool = True):
+                 pad_values: bool = False, chunk: Optional[int] = None, rotary_layout: str = "half", own_kv: bool = True,
+                 head_gate_scope: str = "head"):
         if num_heads % num_kv_heads != 0:
             raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
         if rotary_layout not in ("half", "interleaved"):
@@ -71,6 +75,10 @@ class GQAAttention(Mixer):
         self.names = tuple(names)
         self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
         self.head_gate = head_gate
+        if head_gate_scope not in ("head", "channel"):
+            raise ValueError(f"head_gate_scope '{head_gate_scope}' (head, channel)")
+        self.gate_per_channel = head_gate_scope == "channel"
+        self.gate_size = 0 if head_gate is None else num_heads * (self.value_dim if self.gate_per_channel else 1)
         if qk_norm_scope not in ("head", "all"):
             raise ValueError(f"qk_norm_scope '{qk_norm_scope}' (head, all)")
         if value_mix not in (None, "source", "mix"):
@@ -145,7 +153,7 @@ class GQAAttention(Mixer):
             if self.own_kv:
                 specs[p + k + ".norm"] = TensorSpec((self.kv_size if whole else self.head_dim,))
         if self.head_gate is not None:
-            specs[p + self.head_gate] = TensorSpec((self.num_heads, self.hidden))
+            specs[p + self.head_gate] = TensorSpec((self.gate_size, self.hidden))
         if self.sink == "learned":
             specs[p + "sink"] = TensorSpec((self.num_heads,))
         if self.value_mix is not None:
@@ -187,7 +195,7 @@ class GQAAttention(Mixer):
         if self.qkv_bias:
             bias = [tensors[self._bias_name(i)] if i == 2 else turned(tensors[self._bias_name(i)]) for i in parts]
             if self.head_gate is not None:
-                bias.append(torch.zeros(self.num_heads))
+                bias.append(torch.zeros(self.gate_size))
             self.b_qkv = torch.cat(bias, dim=0).to(torch.float32).to(device).contiguous()
         self.w_o = tensors[p + self.names[3]].to(self.dtype).to(device).contiguous()
         if self.out_bias:
@@ -225,11 +233,15 @@ class GQAAttention(Mixer):
         return self.w_qkv_paired is not None
 
     def weight_bytes(self) -> int:
-        n = self.w_qkv.numel() * self.w_qkv.element_size() + self.w_o.numel() * self.w_o.element_size()
+        n = sum(m.numel() * m.element_size() for m in (self.w_qkv, self.w_o) if m is not None)
         return n + sum(b.numel() * 4 for b in (self.b_qkv, self.b_o) if b is not None)
 
     def out_weight(self) -> torch.Tensor:
         return self.w_o
+
+    def drop_out_weight(self) -> None:
+        """The output matrix has gone into a larger one (see `ParallelBlock`)."""
+        self.w_o = None
 
     def cache_spec(self) -> Optional[PagedKVSpec]:
         if not self.own_kv:
@@ -303,10 +315,10 @@ class GQAAttention(Mixer):
         k.paged_attention(q, ctx.batch, ctx.kv, attn, self.num_heads, self.scale, ws, **more)
         if not direct:
             gate = (qkv, self.q_size + (self.kv_size + self.v_size if self.own_kv else 0)) if self.head_gate is not None else None
-            if padded:
-                k.head_gate(attn, gate, self.num_heads, self.value_dim, scale, out, out_col, x_head_stride=self.value_store)
-            else:
-                k.head_gate(attn, gate, self.num_heads, self.value_dim, scale, out, out_col)
+            extra = {"x_head_stride": self.value_store} if padded else {}
+            if gate is not None and self.gate_per_channel:
+                extra["per_channel"] = True
+            k.head_gate(attn, gate, self.num_heads, self.value_dim, scale, out, out_col, **extra)
 
     def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
         T = x.shape[0]

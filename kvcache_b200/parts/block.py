@@ -156,6 +156,62 @@ class SandwichBlock(Block):
         return NormedDelta(self.ffn.forward(x, ctx), self.post2, gate)
 
 
+class ParallelBlock(Block):
+    """x = norm(h); h += gain * (mixer(x) + ffn(x)): one norm, and both sublayers read its rows.
+
+    Mixer and feed-forward hand over what their last matrices multiply (`forward_heads`, `forward_hidden`) side by side in one
+    buffer, and one product with [Wo | Wdown] makes the sum, which is thus rounded once.  `gain` multiplies the sum in float32
+    where it is added (`ScaledDelta`).  `ffn` may be None."""
+
+    def __init__(self, width: int, norm: Norm, mixer: Mixer, ffn: Optional[FeedForward], dtype: str, gain: float = 1.0):
+        for part, needs in ((mixer, ("forward_heads", "out_weight", "drop_out_weight")), (ffn, ("forward_hidden", "out_weight", "drop_out_weight"))):
+            if part is not None and not all(hasattr(part, name) for name in needs):
+                raise ValueError(f"{type(part).__name__} cannot share its last product with another sublayer ({', '.join(needs)})")
+        self.width, self.norm, self.mixer, self.ffn = width, norm, mixer, ffn
+        self.gain_value = float(gain)
+        self.dtype = TORCH_DTYPES[dtype]
+        self.w_out: Optional[torch.Tensor] = None
+        self.gain: Optional[torch.Tensor] = None
+
+    def _parts(self):
+        return tuple(p for p in (self.norm, self.mixer, self.ffn) if p is not None)
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        out: Dict[str, TensorSpec] = {}
+        for part in self._parts():
+            out.update(part.tensor_specs())
+        return out
+
+    def init_kinds(self) -> Dict[str, str]:
+        out: Dict[str, str] = {}
+        for part in self._parts():
+            out.update(part.init_kinds())
+        return out
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
+        for part in self._parts():
+            part.bind(tensors, device)
+        self.w_out = torch.cat([part.out_weight() for part in self._parts()[1:]], dim=1).contiguous()
+        for part in self._parts()[1:]:
+            part.drop_out_weight()
+        self.gain = None if self.gain_value == 1.0 else torch.full((self.width,), self.gain_value, dtype=torch.float32, device=device)
+
+    def weight_bytes(self) -> int:
+        return sum(part.weight_bytes() for part in self._parts()) + self.w_out.numel() * self.w_out.element_size()
+
+    def forward(self, h: torch.Tensor, pending, ctx: LayerContext):
+        T = h.shape[0]
+        x = ctx.workspace.buffer("block.normed", (T, self.width), self.dtype)
+        self.norm.add_norm(h, pending, x, ctx)
+        both = ctx.workspace.buffer("block.parallel", (T, self.w_out.shape[1]), self.dtype)
+        self.mixer.forward_heads(x, ctx, both)
+        if self.ffn is not None:
+            self.ffn.forward_hidden(x, ctx, both, self.mixer.heads_width)
+        delta = ctx.workspace.buffer("attn.delta", (T, self.width), self.dtype)
+        ctx.kernels.linear(both, self.w_out, delta)
+        return delta if self.gain is None else ScaledDelta(delta, self.gain)
+
+
 class ResidualGate(Part):
     """Logits of a gate on a sublayer's result: W x + b, one number per residual channel, in the compute type.  The
     sigmoid and the multiplication happen where the result is normalised and added (`NormedDelta.gate`)."""

@@ -87,11 +87,18 @@ class GatedMLP(FeedForward):
         return delta
 
 
-class ReluSquaredMLP(FeedForward):
-    """delta = Wdown relu(Wup x)^2; no biases, no gate."""
+PLAIN_ACTIVATIONS = ("relu2", "gelu")
 
-    def __init__(self, hidden: int, intermediate: int, *, prefix: str, dtype: str, names: Sequence[str] = ("up", "down")):
-        self.hidden, self.intermediate = hidden, intermediate
+
+class PlainMLP(FeedForward):
+    """delta = Wdown act(Wup x); no biases, no gate.  act is "relu2": relu(z)^2, or "gelu": z Phi(z) with the normal
+    distribution function."""
+
+    def __init__(self, hidden: int, intermediate: int, *, activation: str, prefix: str, dtype: str, names: Sequence[str] = ("up", "down")):
+        if activation not in PLAIN_ACTIVATIONS:
+            raise ValueError(f"activation '{activation}' is not supported by the plain feed-forward")
+        self.hidden, self.intermediate, self.activation = hidden, intermediate, activation
+        self.hidden_width = intermediate                     # what the matrix on the way down multiplies
         self.prefix, self.names = prefix, tuple(names)
         self.dtype = TORCH_DTYPES[dtype]
         self.w_up: Optional[torch.Tensor] = None
@@ -107,17 +114,37 @@ class ReluSquaredMLP(FeedForward):
         self.w_down = tensors[self.prefix + self.names[1]].to(self.dtype).to(device).contiguous()
 
     def weight_bytes(self) -> int:
-        return (self.w_up.numel() + self.w_down.numel()) * self.w_down.element_size()
+        return sum(m.numel() * m.element_size() for m in (self.w_up, self.w_down) if m is not None)
+
+    def out_weight(self) -> torch.Tensor:
+        return self.w_down
+
+    def drop_out_weight(self) -> None:
+        """The way down has gone into a larger matrix (see `ParallelBlock`)."""
+        self.w_down = None
+
+    def forward_hidden(self, x: torch.Tensor, ctx: LayerContext, out: torch.Tensor, out_col: int = 0) -> None:
+        """act(Wup x) into columns out_col .. out_col + hidden_width of `out`."""
+        act = ctx.workspace.buffer("ffn.act", (x.shape[0], self.intermediate), self.dtype)
+        ctx.kernels.linear(x, self.w_up, act)
+        ctx.kernels.activation_into(act, self.activation, out, out_col)
 
     def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
         T = x.shape[0]
         k, ws = ctx.kernels, ctx.workspace
         act = ws.buffer("ffn.act", (T, self.intermediate), self.dtype)
         k.linear(x, self.w_up, act)
-        k.activation_(act, "relu2")
+        k.activation_(act, self.activation)
         delta = ws.buffer("ffn.delta", (T, self.hidden), self.dtype)
         k.linear(act, self.w_down, delta)
         return delta
+
+
+class ReluSquaredMLP(PlainMLP):
+    """delta = Wdown relu(Wup x)^2; no biases, no gate."""
+
+    def __init__(self, hidden: int, intermediate: int, *, prefix: str, dtype: str, names: Sequence[str] = ("up", "down")):
+        super().__init__(hidden, intermediate, activation="relu2", prefix=prefix, dtype=dtype, names=names)
 
 
 ROUTED_ACTIVATIONS = ("relu2", "clamped_swiglu", "swiglu")

@@ -38,6 +38,22 @@ class RampScaling:
         return 0.1 * math.log(self.factor) + 1.0
 
 
+class LinearScaling:
+    """Slows every pair of a rotation by `factor`; cos and sin keep their size."""
+
+    def __init__(self, factor: float):
+        self.factor = float(factor)
+
+    def key(self) -> tuple:
+        return (self.factor,)
+
+    def blend(self, freq: np.ndarray, dims: int, base: float) -> np.ndarray:
+        return freq / self.factor
+
+    def gain(self) -> float:
+        return 1.0
+
+
 class WavelengthScaling:
     """Slows the pairs of a rotation by their wavelength l = 2 pi / f against the `original` context: pairs with
     l < original / high keep f, pairs with l > original / low turn at f / factor, and between the two the frequency is
@@ -70,7 +86,7 @@ class RotaryHalf(PositionEncoding):
 
     def __init__(self, rotary_dim: int, theta: float, max_positions: int, scaling=None):
         """`scaling`: None, or an object with `blend(freq, dims, base) -> freq` and `gain()` (`RampScaling`,
-        `WavelengthScaling`)."""
+        `LinearScaling`, `WavelengthScaling`)."""
         if rotary_dim % 2 != 0 or rotary_dim < 2:
             raise ValueError(f"rotary_dim must be even and positive, got {rotary_dim}")
         self.rotary_dim = rotary_dim

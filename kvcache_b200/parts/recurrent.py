@@ -262,6 +262,189 @@ class DeltaRuleMixer(_MatrixStateMixer):
         k.head_norm_gate(o, self.norm, self.eps, (proj, self.g_col), "sigmoid", scale, out, out_col, self.num_heads, self.dim)
 
 
+def _padded_rows(t: torch.Tensor, multiple: int) -> torch.Tensor:
+    """`t` with zero rows after its own up to a multiple of `multiple` (products of such sizes start their rows on 16 bytes)."""
+    short = -t.shape[0] % multiple
+    return t if not short else torch.cat([t, torch.zeros(short, t.shape[1], dtype=t.dtype)], dim=0)
+
+
+def _taps_first(weights) -> torch.Tensor:
+    """Convolution weights [channels, taps] of several projections as one float32 [taps, channels]."""
+    return torch.cat([w.to(torch.float32) for w in weights], dim=0).t().contiguous()
+
+
+class GatedDeltaMixer(Mixer):
+    """The gated delta rule with a decay per key channel.  q = Wq h, k = Wk h (num_kv_heads x dim), v = Wv h (num_heads x vdim)
+    each pass a causal convolution of `taps` tokens per channel and silu; q and k become unit vectors x / sqrt(sum x^2 +
+    UNIT_EPS) per head and q is multiplied by dim^(-1/2); query head i reads number i // (num_heads / num_kv_heads) of them.
+    b = sigmoid(Wb h) per head; a = exp(-exp(A_log) softplus(Wa2 Wa1 h + dt_bias)) per head and key channel (A_log per head);
+    S~ = diag(a) S, S = S~ + k (b (v - S~^T k))^T, o = S^T q; each head's o divided by its root mean square, times a weight of
+    vdim numbers that the heads share, times sigmoid(Wg2 Wg1 h); then the output matrix.
+
+    State: the matrices [head, key channel, value channel] and the last taps - 1 inputs of the convolutions, float32.  What
+    enters the recurrence is float32: the projections are written as float32 rows, everything after them is computed from
+    those.  The two low-rank maps run as two products: [Wa1; Wg1] first, then both second factors as the blocks of one
+    matrix (the zeros beside them add nothing)."""
+
+    UNIT_EPS = 1e-6
+
+    def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, taps: int, *, eps: float, prefix: str,
+                 dtype: str, decay_rank: Optional[int] = None, gate_rank: Optional[int] = None):
+        if num_heads % num_kv_heads != 0:
+            raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
+        self.hidden, self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.taps = hidden, num_heads, num_kv_heads, dim, vdim, taps
+        self.decay_rank, self.gate_rank = decay_rank, gate_rank      # None: whatever the checkpoint's two factors agree on
+        self.eps, self.prefix = float(eps), prefix
+        self.dtype = TORCH_DTYPES[dtype]
+        self.qk_size, self.heads_width, self.decay_size = num_kv_heads * dim, num_heads * vdim, num_heads * dim
+        self.channels = 2 * self.qk_size + self.heads_width          # what the convolutions run over: [q | k | v]
+        self.q_scale = 1.0 / math.sqrt(dim)
+        self.w_in = self.w_low = self.w_high = self.w_o = None
+        self.conv_w = self.dt_bias = self.rate = self.norm = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        p, W = self.prefix, self.hidden
+        specs = {}
+        for name, size in (("q", self.qk_size), ("k", self.qk_size), ("v", self.heads_width)):
+            specs[p + name] = TensorSpec((size, W))
+            specs[p + name + ".conv"] = TensorSpec((size, self.taps))
+        specs.update({p + "b": TensorSpec((self.num_heads, W)), p + "A_log": TensorSpec((self.num_heads,)), p + "norm": TensorSpec((self.vdim,)),
+                      p + "a1": TensorSpec((self.decay_rank, W)), p + "a2": TensorSpec((self.decay_size, self.decay_rank)),
+                      p + "dt_bias": TensorSpec((self.decay_size,)), p + "g1": TensorSpec((self.gate_rank, W)),
+                      p + "g2": TensorSpec((self.heads_width, self.gate_rank)), p + "o": TensorSpec((W, self.heads_width))})
+        return specs
+
+    def init_kinds(self) -> Dict[str, str]:
+        return {self.prefix + "norm": "ones_plus_normal"}
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
+        p = self.prefix
+        place = lambda t: t.to(self.dtype).to(device).contiguous()
+        plain = lambda t: t.to(torch.float32).to(device).contiguous()
+        for one, two in (("a1", "a2"), ("g1", "g2")):
+            if tensors[p + one].shape[0] != tensors[p + two].shape[1]:
+                raise WeightError(f"{p}{one} has {tensors[p + one].shape[0]} rows but {p}{two} has {tensors[p + two].shape[1]} columns")
+        self.w_in = place(_padded_rows(torch.cat([tensors[p + n] for n in ("q", "k", "v", "b")], dim=0), 8))
+        self.w_low = place(_padded_rows(torch.cat([tensors[p + "a1"], tensors[p + "g1"]], dim=0), 32))
+        a2, g2 = tensors[p + "a2"], tensors[p + "g2"]
+        high = torch.zeros(a2.shape[0] + g2.shape[0], self.w_low.shape[0], dtype=a2.dtype)
+        high[:a2.shape[0], :a2.shape[1]] = a2
+        high[a2.shape[0]:, a2.shape[1]:a2.shape[1] + g2.shape[1]] = g2
+        self.w_high = place(high)
+        self.w_o = place(tensors[p + "o"])
+        self.conv_w = _taps_first([tensors[p + n + ".conv"] for n in ("q", "k", "v")]).to(device)
+        self.dt_bias, self.norm = plain(tensors[p + "dt_bias"]), plain(tensors[p + "norm"])
+        self.rate = plain(torch.exp(tensors[p + "A_log"].to(torch.float64)))
+
+    def weight_bytes(self) -> int:
+        return sum(m.numel() * m.element_size() for m in (self.w_in, self.w_low, self.w_high, self.w_o) if m is not None)
+
+    def out_weight(self) -> torch.Tensor:
+        return self.w_o
+
+    def drop_out_weight(self) -> None:
+        self.w_o = None
+
+    def state_spec(self):
+        return {"memory": StateSpec((self.num_heads, self.dim, self.vdim)), "conv": StateSpec((self.taps - 1, self.channels))}
+
+    def forward_heads(self, x: torch.Tensor, ctx: LayerContext, out: torch.Tensor, out_col: int = 0, scale: float = 1.0) -> None:
+        T, H, G, D, V = x.shape[0], self.num_heads, self.num_kv_heads, self.dim, self.vdim
+        k, ws = ctx.kernels, ctx.workspace
+        proj = ws.buffer("recurrent.proj", (T, self.w_in.shape[0]), torch.float32)
+        k.linear(x, self.w_in, proj)
+        low = ws.buffer("recurrent.low", (T, self.w_low.shape[0]), self.dtype)
+        k.linear(x, self.w_low, low)
+        z = ws.buffer("recurrent.z", (T, self.decay_size + self.heads_width), torch.float32)      # [decay logits | gate logits]
+        k.linear(low, self.w_high, z)
+        rows = ws.buffer("recurrent.rows", (T, self.channels), torch.float32)
+        gates = ws.buffer("recurrent.gates", (T, self.decay_size + H), torch.float32)
+        k.gated_delta_inputs(proj, self.channels, self.conv_w, ctx.state["conv"], z, self.dt_bias, self.rate, self.UNIT_EPS, ctx.batch,
+                             rows, gates, H, G, D, V)
+        o = ws.buffer("recurrent.o", (T, self.heads_width), torch.float32)
+        k.gated_delta_scan(rows, gates, self.q_scale, ctx.batch, ctx.state["memory"], o, H, G, D, V, ws)
+        k.head_norm_gate(o, self.norm, self.eps, (z, self.decay_size), "sigmoid", scale, out, out_col, H, V)
+
+    def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
+        gated = ctx.workspace.buffer("recurrent.gated", (x.shape[0], self.heads_width), self.dtype)
+        self.forward_heads(x, ctx, gated)
+        delta = ctx.workspace.buffer("attn.delta", (x.shape[0], self.hidden), self.dtype)
+        ctx.kernels.linear(gated, self.w_o, delta)
+        return delta
+
+
+class StateSpaceMixer(Mixer):
+    """A selective state space with one decay per head.  Win h = [z: inner | x: inner | B: groups * state | C: groups * state |
+    dt: num_heads], inner = num_heads * vdim; x, B and C pass a causal convolution of `taps` tokens per channel, with a bias,
+    and silu; d = softplus(dt + dt_bias); with the group i // (num_heads / groups) of head i,
+    S = exp(-exp(A_log) d) S + d B x^T, y = S^T C + D x; y silu(z) (the gate first), in `norm_parts` equal parts each divided
+    by its own root mean square, times a weight of inner numbers; then the output matrix.  State: the matrices
+    [head, state, value channel] and the last taps - 1 inputs of the convolution, float32."""
+
+    def __init__(self, hidden: int, num_heads: int, vdim: int, state: int, groups: int, norm_parts: int, taps: int, *, eps: float,
+                 prefix: str, dtype: str):
+        if num_heads % groups != 0 or (num_heads * vdim) % norm_parts != 0:
+            raise ValueError(f"{num_heads} heads of {vdim}: {groups} groups and {norm_parts} parts of the norm must divide them evenly")
+        self.hidden, self.num_heads, self.vdim, self.state, self.groups = hidden, num_heads, vdim, state, groups
+        self.norm_parts, self.taps = norm_parts, taps
+        self.eps, self.prefix = float(eps), prefix
+        self.dtype = TORCH_DTYPES[dtype]
+        self.heads_width = num_heads * vdim
+        self.channels = self.heads_width + 2 * groups * state            # what the convolution runs over: [x | B | C]
+        self.w_in = self.w_o = None
+        self.conv_w = self.conv_b = self.dt_bias = self.rate = self.skip = self.norm = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        p, H = self.prefix, self.num_heads
+        return {p + "in": TensorSpec((self.heads_width + self.channels + H, self.hidden)), p + "conv": TensorSpec((self.channels, self.taps)),
+                p + "conv.b": TensorSpec((self.channels,)), p + "dt_bias": TensorSpec((H,)), p + "A_log": TensorSpec((H,)),
+                p + "D": TensorSpec((H,)), p + "norm": TensorSpec((self.heads_width,)), p + "o": TensorSpec((self.hidden, self.heads_width))}
+
+    def init_kinds(self) -> Dict[str, str]:
+        return {self.prefix + "norm": "ones_plus_normal"}
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], device: torch.device) -> None:
+        p = self.prefix
+        plain = lambda name: tensors[p + name].to(torch.float32).to(device).contiguous()
+        self.w_in = _padded_rows(tensors[p + "in"], 8).to(self.dtype).to(device).contiguous()
+        self.w_o = tensors[p + "o"].to(self.dtype).to(device).contiguous()
+        self.conv_w = _taps_first([tensors[p + "conv"]]).to(device)
+        self.conv_b, self.dt_bias, self.skip, self.norm = plain("conv.b"), plain("dt_bias"), plain("D"), plain("norm")
+        self.rate = torch.exp(tensors[p + "A_log"].to(torch.float64)).to(torch.float32).to(device).contiguous()
+
+    def weight_bytes(self) -> int:
+        return sum(m.numel() * m.element_size() for m in (self.w_in, self.w_o) if m is not None)
+
+    def out_weight(self) -> torch.Tensor:
+        return self.w_o
+
+    def drop_out_weight(self) -> None:
+        self.w_o = None
+
+    def state_spec(self):
+        return {"memory": StateSpec((self.num_heads, self.state, self.vdim)), "conv": StateSpec((self.taps - 1, self.channels))}
+
+    def forward_heads(self, x: torch.Tensor, ctx: LayerContext, out: torch.Tensor, out_col: int = 0, scale: float = 1.0) -> None:
+        T, H, W = x.shape[0], self.num_heads, self.heads_width
+        k, ws = ctx.kernels, ctx.workspace
+        proj = ws.buffer("recurrent.proj", (T, self.w_in.shape[0]), torch.float32)
+        k.linear(x, self.w_in, proj)
+        rows = ws.buffer("recurrent.rows", (T, self.channels), torch.float32)
+        gates = ws.buffer("recurrent.gates", (T, 2 * H), torch.float32)
+        k.state_space_inputs(proj, W, W + self.channels, self.conv_w, self.conv_b, ctx.state["conv"], self.dt_bias, self.rate, ctx.batch,
+                             rows, gates, H)
+        y = ws.buffer("recurrent.o", (T, W), torch.float32)
+        k.state_space_scan(rows, gates, ctx.batch, ctx.state["memory"], y, H, self.groups, self.state, self.vdim, ws)
+        k.gate_part_norm(y, rows, self.skip, (proj, 0), self.norm, self.eps, scale, out, out_col, H, self.vdim, self.norm_parts)
+
+    def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
+        gated = ctx.workspace.buffer("recurrent.gated", (x.shape[0], self.heads_width), self.dtype)
+        self.forward_heads(x, ctx, gated)
+        delta = ctx.workspace.buffer("attn.delta", (x.shape[0], self.hidden), self.dtype)
+        ctx.kernels.linear(gated, self.w_o, delta)
+        return delta
+
+
 class ParallelMixer(Mixer):
     """Two mixers side by side on the same rows: delta = left_scale * left(x) + right_scale * right(x).
 
@@ -277,6 +460,7 @@ class ParallelMixer(Mixer):
             raise ValueError("only one side of a parallel mixer may keep keys and values in pages")
         self.hidden = hidden
         self.left, self.right = left, right
+        self.heads_width = left.heads_width + right.heads_width
         self.left_scale, self.right_scale = float(left_scale), float(right_scale)
         self.dtype = TORCH_DTYPES[dtype]
         self.w_o: Optional[torch.Tensor] = None
@@ -321,12 +505,20 @@ class ParallelMixer(Mixer):
         return LayerContext(batch=ctx.batch, kernels=ctx.kernels, workspace=ctx.workspace, kv=ctx.kv, state=state,
                             call_index=ctx.call_index, embedded=ctx.embedded)
 
+    def out_weight(self) -> torch.Tensor:
+        return self.w_o
+
+    def drop_out_weight(self) -> None:
+        self.w_o = None
+
+    def forward_heads(self, x: torch.Tensor, ctx: LayerContext, out: torch.Tensor, out_col: int = 0, scale: float = 1.0) -> None:
+        self.left.forward_heads(x, self._side_context(ctx, self.left.state_spec(), "left"), out, out_col, scale * self.left_scale)
+        self.right.forward_heads(x, self._side_context(ctx, self.right.state_spec(), "right"), out, out_col + self.left.heads_width,
+                                 scale * self.right_scale)
+
     def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
-        T = x.shape[0]
-        wl = self.left.heads_width
-        both = ctx.workspace.buffer("parallel.heads", (T, wl + self.right.heads_width), self.dtype)
-        self.left.forward_heads(x, self._side_context(ctx, self.left.state_spec(), "left"), both, 0, self.left_scale)
-        self.right.forward_heads(x, self._side_context(ctx, self.right.state_spec(), "right"), both, wl, self.right_scale)
-        delta = ctx.workspace.buffer("attn.delta", (T, self.hidden), self.dtype)
+        both = ctx.workspace.buffer("parallel.heads", (x.shape[0], self.heads_width), self.dtype)
+        self.forward_heads(x, ctx, both)
+        delta = ctx.workspace.buffer("attn.delta", (x.shape[0], self.hidden), self.dtype)
         ctx.kernels.linear(both, self.w_o, delta)
         return delta

@@ -376,13 +376,16 @@ class TorchKernels:
                 h[r] += table[row].to(torch.float32)
             previous[slot] = int(ids[lo + n - 1])
 
-    def head_gate(self, x, gate, num_heads, value_dim, scale, out, out_col=0, x_head_stride=None):
+    def head_gate(self, x, gate, num_heads, value_dim, scale, out, out_col=0, x_head_stride=None, per_channel=False):
         f = self.f
         T = x.shape[0]
         y = x.to(f).view(T, num_heads, x_head_stride or value_dim)[:, :, :value_dim]
         if gate is not None:
             src, col = gate
-            y = y * torch.sigmoid(src[:, col:col + num_heads].to(f))[:, :, None]
+            if per_channel:
+                y = y * torch.sigmoid(src[:, col:col + num_heads * value_dim].to(f)).view(T, num_heads, value_dim)
+            else:
+                y = y * torch.sigmoid(src[:, col:col + num_heads].to(f))[:, :, None]
         out[:, out_col:out_col + num_heads * value_dim] = (y * scale).reshape(T, -1).to(out.dtype)
 
     def head_norm_gate(self, o, weight, eps, gate, activation, scale, out, out_col, num_heads, value_dim, scope="head"):
@@ -468,7 +471,86 @@ class TorchKernels:
 
     def activation_(self, x, kind, cap=0.0):
         v = x.to(self.f)
-        x.copy_((torch.tanh(v) if kind == "tanh" else torch.relu(v) ** 2 if kind == "relu2" else cap * torch.tanh(v / cap)).to(x.dtype))
+        x.copy_(self._activated(v, kind, cap).to(x.dtype))
+
+    @staticmethod
+    def _activated(v, kind, cap):
+        if kind == "gelu":
+            return 0.5 * v * (1.0 + torch.erf(v / 2.0 ** 0.5))
+        return torch.tanh(v) if kind == "tanh" else torch.relu(v) ** 2 if kind == "relu2" else cap * torch.tanh(v / cap)
+
+    def activation_into(self, x, kind, out, out_col=0, cap=0.0):
+        out[:, out_col:out_col + x.shape[1]] = self._activated(x.to(self.f), kind, cap).to(out.dtype)
+
+    # ---- operators of the short convolutions, the gated delta rule and the state-space mixer ------------------------------
+    def _short_conv(self, x, conv_w, conv_b, tail, batch):
+        """silu(bias + sum_n w[n] x_{t - (taps - 1) + n}) per segment; tail[slot] holds the inputs before the segment's first."""
+        f = self.f
+        taps = conv_w.shape[0]
+        out = torch.empty(x.shape, dtype=f)
+        for lo, n, slot in self._segments(batch):
+            seq = torch.cat([tail[slot].to(f), x[lo:lo + n].to(f)], dim=0)
+            y = sum(conv_w[j].to(f) * seq[j:j + n] for j in range(taps))
+            if conv_b is not None:
+                y = y + conv_b.to(f)
+            out[lo:lo + n] = y * torch.sigmoid(y)
+            if taps > 1:
+                tail[slot] = seq[-(taps - 1):].to(tail.dtype)
+        return out
+
+    def gated_delta_inputs(self, proj, b_col, conv_w, tail, z, dt_bias, rate, unit_eps, batch, rows, gates, H, G, D, Dv):
+        f = self.f
+        T = proj.shape[0]
+        y = self._short_conv(proj[:, :2 * G * D + H * Dv], conv_w, None, tail, batch)
+        qk = y[:, :2 * G * D].view(T, 2 * G, D)
+        qk = qk / torch.sqrt((qk * qk).sum(dim=-1, keepdim=True) + unit_eps)
+        rows.copy_(torch.cat([qk.reshape(T, -1), y[:, 2 * G * D:]], dim=1).to(rows.dtype))
+        soft = torch.nn.functional.softplus(z[:, :H * D].to(f) + dt_bias.to(f), threshold=1e9).view(T, H, D)
+        decay = torch.exp(-rate.to(f)[None, :, None] * soft)
+        gates.copy_(torch.cat([decay.reshape(T, -1), torch.sigmoid(proj[:, b_col:b_col + H].to(f))], dim=1).to(gates.dtype))
+
+    def gated_delta_scan(self, rows, gates, q_scale, batch, memory, out, H, G, D, Dv, workspace=None):
+        f = self.f
+        shared = torch.arange(H) // (H // G)
+        for lo, n, slot in self._segments(batch):
+            S = memory[slot].to(f)
+            for t in range(lo, lo + n):
+                q, k = (rows[t, c:c + G * D].to(f).view(G, D)[shared] for c in (0, G * D))
+                v = rows[t, 2 * G * D:].to(f).view(H, Dv)
+                S = gates[t, :H * D].to(f).view(H, D)[:, :, None] * S
+                u = gates[t, H * D:].to(f)[:, None] * (v - torch.einsum("hkv,hk->hv", S, k))
+                S = S + k[:, :, None] * u[:, None, :]
+                out[t] = (q_scale * torch.einsum("hkv,hk->hv", S, q)).reshape(-1).to(out.dtype)
+            memory[slot] = S.to(memory.dtype)
+
+    def state_space_inputs(self, proj, col, dt_col, conv_w, conv_b, tail, dt_bias, rate, batch, rows, gates, H):
+        f = self.f
+        rows.copy_(self._short_conv(proj[:, col:col + conv_w.shape[1]], conv_w, conv_b, tail, batch).to(rows.dtype))
+        d = torch.nn.functional.softplus(proj[:, dt_col:dt_col + H].to(f) + dt_bias.to(f), threshold=1e9)
+        gates.copy_(torch.cat([torch.exp(-rate.to(f) * d), d], dim=1).to(gates.dtype))
+
+    def state_space_scan(self, rows, gates, batch, memory, out, H, G, N, Dv, workspace=None):
+        f = self.f
+        shared = torch.arange(H) // (H // G)
+        for lo, n, slot in self._segments(batch):
+            S = memory[slot].to(f)
+            for t in range(lo, lo + n):
+                x = rows[t, :H * Dv].to(f).view(H, Dv)
+                B, C = (rows[t, c:c + G * N].to(f).view(G, N)[shared] for c in (H * Dv, H * Dv + G * N))
+                keep, d = gates[t, :H].to(f), gates[t, H:].to(f)
+                S = keep[:, None, None] * S + d[:, None, None] * B[:, :, None] * x[:, None, :]
+                out[t] = torch.einsum("hnv,hn->hv", S, C).reshape(-1).to(out.dtype)
+            memory[slot] = S.to(memory.dtype)
+
+    def gate_part_norm(self, o, x, skip, gate, weight, eps, scale, out, out_col, num_heads, value_dim, parts):
+        f = self.f
+        T, W = o.shape
+        src, col = gate
+        g = src[:, col:col + W].to(f)
+        y = (o.to(f) + skip.to(f).repeat_interleave(value_dim) * x[:, :W].to(f)) * (g * torch.sigmoid(g))
+        y = y.view(T, parts, -1)
+        y = (y * torch.rsqrt((y * y).mean(dim=-1, keepdim=True) + eps)).reshape(T, W)
+        out[:, out_col:out_col + W] = (y * weight.to(f) * scale).to(out.dtype)
 
     def delta_rule_scan(self, proj, cols, z, rate, unit_eps, batch, memory, out, H, D, workspace=None):
         """Per segment, from and into memory[slot] ([H, D, D]): w = exp(-rate sigmoid(z)), a = sigmoid(proj[a_col]),
