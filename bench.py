@@ -1,7 +1,7 @@
 """Benchmark of kvcache_b200: decode tokens a second of the Qwen2.5-0.5B shape on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-    python bench.py --design kakipel|libulorn|lipelix|karorax|kunulorn [--sizes 0.5B-like,3B-like]     (another workload, see `run_design`; the default stays as it is)
+    python bench.py --design kakipel|libulorn|lipelix|karorax|kunulorn|kaposun [--sizes 0.5B-like,3B-like]     (another workload, see `run_design`; the default stays as it is)
 
 One JSON line on standard output.  `value`: decoded tokens a second at batch 8 and the
 benchmark context (device-timed decode steps through the engine's step function and device
@@ -547,6 +547,31 @@ def kunulorn_sizes():
     return out
 
 
+def kaposun_sizes():
+    """Layer sizes that resemble real models, as (name, {architecture: config}): a Kaposun model of four layers (attention over
+    all keys; parallel: window attention that keeps the first tokens beside the gated delta rule; a state space; parallel; every
+    layer with the plain feed-forward), beside the Lipelix, Libulorn and Qwen2 models of `lipelix_sizes` at equal width, heads,
+    feed-forward width and vocabulary: Lipelix has the closest delta rule, window attention and plain feed-forward, Libulorn the
+    closest parallel layer."""
+    out = []
+    others = dict(lipelix_sizes())
+    for name, width, heads, kv_heads, dim, d_heads, d_dim, rank, s_heads, s_vdim, state, ff, vocab in (
+            ("0.5B-like", 896, 14, 2, 64, 14, 64, 64, 28, 64, 128, 4864, 32768),
+            ("3B-like", 2048, 16, 2, 128, 16, 128, 128, 64, 64, 128, 11008, 32768)):
+        common = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+        full = {"type": "attention", "mixer": dict(common, rot={"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 4.0}})}
+        right = {"heads": d_heads, "kv_heads": d_heads, "dim": d_dim, "vdim": d_dim, "conv": 4, "decay_rank": rank, "gate_rank": rank}
+        parallel = {"type": "parallel", "mixer": {"left": dict(common, mask={"size": 1024, "keep_first": 4}), "right": right,
+                                                  "left_scale": 1.0, "right_scale": 1.0}}
+        space = {"type": "mamba2", "mixer": {"heads": s_heads, "vdim": s_vdim, "state": state, "groups": 1, "norm_groups": 1, "conv": 4}}
+        mlp = {"kind": "dense", "ff": ff}
+        kap = {"architecture": "Kaposun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+               "layers": [dict(layer, mlp=mlp) for layer in (full, parallel, space, parallel)], "initializer_range": 0.02}
+        out.append((name, {"kaposun": kap, "lipelix": others[name]["lipelix"], "libulorn": others[name]["libulorn"],
+                           "qwen2": others[name]["qwen2"]}))
+    return out
+
+
 def _write_design_folder(tmp, tag, config):
     import torch
     import kvcache_b200  # noqa: F401
@@ -639,7 +664,7 @@ def _time_classes(folder, peaks, mode, batch, context, tokens, repeats=3):
 
 
 def run_design(args) -> int:
-    """`--design kakipel | libulorn | lipelix | karorax | kunulorn`: decode and prefill throughput of that architecture at sizes that resemble real models'
+    """`--design kakipel | libulorn | lipelix | karorax | kunulorn | kaposun`: decode and prefill throughput of that architecture at sizes that resemble real models'
     layers, beside the Qwen2 architecture at equal width, layer runs, feed-forward width and vocabulary (random weights,
     random cache contents for decode), and every class of kernel of one step of each against its roofline."""
     peaks = load_peaks()
@@ -653,6 +678,8 @@ def run_design(args) -> int:
         sizes, beside = karorax_sizes(), "Karorax beside Libulorn, Kakipel and Qwen2"
     elif args.design == "kunulorn":
         sizes, beside = kunulorn_sizes(), "Kunulorn beside Libulorn, Lipelix and Qwen2"
+    elif args.design == "kaposun":
+        sizes, beside = kaposun_sizes(), "Kaposun beside Lipelix, Libulorn and Qwen2"
     else:
         sizes, beside = [(name, {"kakipel": kaki, "qwen2": qwen}) for name, kaki, qwen in design_sizes()], "Kakipel beside Qwen2"
     done = {}
@@ -775,7 +802,7 @@ def main() -> int:
     parser.add_argument("--skip-prefill", action="store_true")
     parser.add_argument("--skip-kernels", action="store_true")
     parser.add_argument("--no-graphs", action="store_true", help="launch the decode step's kernels one by one (for profilers)")
-    parser.add_argument("--design", default=None, choices=["kakipel", "libulorn", "lipelix", "karorax", "kunulorn"],
+    parser.add_argument("--design", default=None, choices=["kakipel", "libulorn", "lipelix", "karorax", "kunulorn", "kaposun"],
                         help="instead of the default workload: this architecture beside Qwen2 at equal sizes (decode, prefill, kernels)")
     parser.add_argument("--sizes", default="", help="with --design: the sizes to run, with commas between them (default: all)")
     args = parser.parse_args()

@@ -49,7 +49,8 @@ class KernelTiming:
     OPERATORS = ("embed", "add_rmsnorm", "silu_mul", "gate_up_act", "linear", "qkv_rope_append", "rope_append_attention",
                  "paged_attention", "sample", "norm_add_rmsnorm", "latent_norm_rope_append", "head_linear", "latent_attention",
                  "route_top", "route_sigmoid", "routed_experts", "bigram_embed", "head_gate", "head_norm_gate", "gated_linear_scan",
-                 "matrix_memory_scan", "token_shift", "activation_", "delta_rule_scan", "lightning_scan")
+                 "matrix_memory_scan", "token_shift", "activation_", "activation_into", "delta_rule_scan", "lightning_scan",
+                 "gated_delta_inputs", "gated_delta_scan", "state_space_inputs", "state_space_scan", "gate_part_norm")
 
     def __init__(self, kernels, hold_ms: float = 4.0):
         self.kernels = kernels
@@ -115,7 +116,7 @@ class KernelTiming:
             h, table = args[3], args[0]
             return name, h.numel() * (8 + table.element_size())
         if name == "head_gate":
-            return name, 2 * _numel_bytes(args[0])
+            return name, (3 if kwargs.get("per_channel") else 2) * _numel_bytes(args[0])
         if name == "head_norm_gate":
             o, out, H, Dv = args[0], args[6], args[8], args[9]
             return name, 2 * _numel_bytes(o) + o.shape[0] * H * Dv * out.element_size()
@@ -139,8 +140,24 @@ class KernelTiming:
         if name == "token_shift":
             x, out = args[0], args[4]
             return name, _numel_bytes(x) + _numel_bytes(out)
-        if name == "activation_":
-            return name, 2 * _numel_bytes(args[0])
+        if name in ("activation_", "activation_into"):
+            return "activation", 2 * _numel_bytes(args[0])
+        if name == "gated_delta_inputs":
+            # The projections, the decay logits, the convolutions' states in and out; the rows and gates out.
+            tail, z, batch, rows, gates, H, D = args[3], args[4], args[8], args[9], args[10], args[11], args[13]
+            return name, 2 * _numel_bytes(rows) + _numel_bytes(gates) + 4 * z.shape[0] * (H * D + H) + 8 * batch.num_segments * tail[0].numel()
+        if name == "gated_delta_scan":
+            rows, gates, batch, out, H, D, Dv = args[0], args[1], args[3], args[5], args[6], args[8], args[9]
+            return f"{name} {H}x{D}x{Dv}", _numel_bytes(rows) + _numel_bytes(gates) + _numel_bytes(out) + 8 * batch.num_segments * H * D * Dv
+        if name == "state_space_inputs":
+            tail, batch, rows, gates = args[5], args[8], args[9], args[10]
+            return name, 2 * _numel_bytes(rows) + 2 * _numel_bytes(gates) + 8 * batch.num_segments * tail[0].numel()
+        if name == "state_space_scan":
+            rows, gates, batch, out, H, N, Dv = args[0], args[1], args[2], args[4], args[5], args[7], args[8]
+            return f"{name} {H}x{N}x{Dv}", _numel_bytes(rows) + _numel_bytes(gates) + _numel_bytes(out) + 8 * batch.num_segments * H * N * Dv
+        if name == "gate_part_norm":
+            o, out, H, Dv = args[0], args[7], args[9], args[10]
+            return name, 3 * _numel_bytes(o) + o.shape[0] * H * Dv * out.element_size()
         return name, 0
 
     @staticmethod
@@ -192,6 +209,11 @@ class KernelTiming:
         if name == "delta_rule_scan":
             # per row and state element: decay, the read along the unit key, its removal, the new outer product, read-out
             return 9 * args[0].shape[0] * args[8] * args[9] * args[9]
+        if name == "gated_delta_scan":
+            # per row and state element: decay, the read along the key, the new outer product, read-out
+            return 7 * args[0].shape[0] * args[6] * args[8] * args[9]
+        if name == "state_space_scan":
+            return 4 * args[0].shape[0] * args[5] * args[7] * args[8]
         return 0
 
     # ---- switching on and off -------------------------------------------------------------------------
