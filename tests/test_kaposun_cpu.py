@@ -195,3 +195,333 @@ def test_attention_part_alone(m, gated):
         got.append(part.forward(x[at:at + n], _context(batch, kv)))
         at += n
     assert_close(torch.cat(got), want, 1e-5)
+
+
+def _edge_case(part, W, T, at, strength=40.0, seed=3):
+    """Weights and inputs of an attention part in which every query scores the key of row `at` far above all others: channel 0
+    of the input is 1 in that row only and drives the keys along one direction, channel 1 is 1 in every row and drives the
+    queries along the same direction; channel 2 drives all other rows' keys along another (keys are normalised, and small random
+    ones would point anywhere)."""
+    g = torch.Generator().manual_seed(seed)
+    w = {name: (torch.randn(spec.shape, generator=g) * 0.05 + (1.0 if name.endswith("norm") else 0.0)).to(torch.bfloat16)
+         for name, spec in part.tensor_specs().items()}
+    D = part.head_dim
+    q, k = w["m.q"].float(), w["m.k"].float()
+    q[:, :3], k[:, :3] = 0.0, 0.0
+    q[torch.arange(part.num_heads) * D, 1] = strength
+    k[torch.arange(part.num_kv_heads) * D, 0] = strength
+    k[torch.arange(part.num_kv_heads) * D + 1, 2] = strength
+    w["m.q"], w["m.k"] = q.to(torch.bfloat16), k.to(torch.bfloat16)
+    x = torch.randn(T, W, generator=g) * 0.1
+    x[:, 0], x[:, 1], x[:, 2] = 0.0, 1.0, 1.0
+    x[at, 0], x[at, 2] = 1.0, 0.0
+    return w, x
+
+
+@pytest.mark.parametrize("at,mask,taken", [(0, None, True), (150, (90, 6), True), (149, (90, 6), False), (5, (90, 6), True), (6, (90, 6), False),
+                                            (15, (20, 16), True), (16, (20, 16), False)])
+def test_one_key_far_away_takes_all_the_weight_or_none(at, mask, taken):
+    """Random weights would hide a lost key among hundreds.  Row 239 sees keys 150 .. 239 of a window of 90 and the kept ones."""
+    T, W = 240, 24
+    m = dict(heads=4, kv_heads=2, dim=8, vdim=6, scale=40.0)
+    if mask:
+        m["mask"] = {"size": mask[0], "keep_first": mask[1]}
+    part = _attention_part(W, m)
+    w, x = _edge_case(part, W, T, at)
+    part.bind(w, torch.device("cpu"))
+    wd = {k: v.double() for k, v in w.items()}
+    want = plain.attention(m, wd, "m.", x.double(), torch.arange(T), 1e-5)
+    value = (x[at].double() @ wd["m.v"].t()).view(2, 6).repeat_interleave(2, dim=0).reshape(1, -1) @ wd["m.o"].t()
+    assert bool((want[239] - value).abs().max() < 1e-3 * want.abs().max()) == taken
+    _, kv = _scenario([(0, T)], part.cache_spec(), page_size=16)
+    got, start = [], 0
+    for n in [131, 2, 67, 32] + [1] * 8:
+        batch, _ = _scenario([(start, n)], part.cache_spec(), page_size=16)
+        got.append(part.forward(x[start:start + n], _context(batch, kv)))
+        start += n
+    assert_close(torch.cat(got), want, 1e-5)
+
+
+# The recurrent mixers: (part, plain function of (weights, rows)).
+def _delta_part(W, H, G, D, V, taps, ranks=(6, 5), eps=1e-5):
+    from kvcache_b200.parts.recurrent import GatedDeltaMixer
+    m = {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "conv": taps}
+    part = GatedDeltaMixer(W, H, G, D, V, taps, eps=eps, prefix="m.", dtype="float32", decay_rank=ranks[0], gate_rank=ranks[1])
+    return part, lambda w, x: plain.gated_delta(m, w, "m.", x, eps)
+
+
+def _space_part(W, H, V, N, G, parts, taps, eps=1e-5):
+    from kvcache_b200.parts.recurrent import StateSpaceMixer
+    m = {"heads": H, "vdim": V, "state": N, "groups": G, "norm_groups": parts, "conv": taps}
+    part = StateSpaceMixer(W, H, V, N, G, parts, taps, eps=eps, prefix="m.", dtype="float32")
+    return part, lambda w, x: plain.mamba2(m, w, "m.", x, eps)
+
+
+RECURRENT = {"delta": lambda W: _delta_part(W, 4, 2, 6, 10, 4), "delta, one tap": lambda W: _delta_part(W, 3, 3, 8, 8, 1),
+             "delta, long convolution": lambda W: _delta_part(W, 6, 1, 5, 3, 6, (9, 33)), "space": lambda W: _space_part(W, 4, 6, 5, 2, 3, 4),
+             "space, one tap": lambda W: _space_part(W, 3, 8, 9, 1, 1, 1), "space, a group a head": lambda W: _space_part(W, 5, 4, 7, 5, 10, 2)}
+
+
+@pytest.mark.parametrize("which", list(RECURRENT))
+def test_recurrent_mixer_alone_in_portions_and_beside_others(which):
+    """Whole; one token at a time; portions shorter than the convolution; two requests beside one another in slots whose order is
+    not the segments'; a slot that another request held, zeroed as at admission."""
+    W, T = 20, 31
+    part, reference = RECURRENT[which](W)
+    w = _weights(part.tensor_specs(), 5)
+    part.bind(w, torch.device("cpu"))
+    wd = {k: v.double() for k, v in w.items()}
+    x, other = (torch.randn(T, W, generator=torch.Generator().manual_seed(s)) for s in (6, 7))
+    want, want_other = reference(wd, x.double()), reference(wd, other.double())
+    for name in wd:                                   # every tensor matters
+        assert (reference(dict(wd, **{name: wd[name] * 0.5 + 0.3}), x.double()) - want).abs().max() > 1e-3 * want.abs().max(), name
+    state = _states(part)
+
+    def run(pieces):
+        batch, _ = _scenario([(start, len(rows)) for start, rows, _ in pieces], slots=[slot for _, _, slot in pieces])
+        return part.forward(torch.cat([rows for _, rows, _ in pieces]), _context(batch, state=state)).clone()
+    assert_close(run([(0, x, 1)]), want, 1e-5, "whole")
+    for sizes in ([1] * T, [2, 1, 1, 3, 2, 5, 17]):
+        for s in state.values():
+            s[1].zero_()
+        got, at = [], 0
+        for n in sizes:
+            got.append(run([(at, x[at:at + n], 1)]))
+            at += n
+        assert_close(torch.cat(got), want, 1e-5, f"portions {sizes[:3]}")
+    for s in state.values():
+        s.zero_()
+        s[1].fill_(7.0)                               # nobody's: must stay
+    first = run([(0, x[:9], 2), (0, other[:1], 0)])
+    second = run([(1, other[1:3], 0), (9, x[9:10], 2)])
+    third = run([(10, x[10:], 2), (3, other[3:], 0)])
+    assert_close(torch.cat([first[:9], second[2:], third[:21]]), want, 1e-5, "beside another request")
+    assert_close(torch.cat([first[9:], second[:2], third[21:]]), want_other, 1e-5, "the other request")
+    assert all(bool((s[1] == 7.0).all()) for s in state.values())
+
+
+def test_gated_delta_reads_after_the_decay_and_before_its_own_write():
+    """No convolution, one head, key and query the first unit vector: with write strength b and decay a the state along that key
+    goes s -> a s + b (v - a s), and the read-out sees it; reading the undecayed state, or before the write, differs."""
+    k = TorchKernels(wide=True)
+    batch, _ = _scenario([(0, 3)], slots=[0])
+    D = Dv = 2
+    rows = torch.tensor([[1.0, 0.0, 1.0, 0.0, 5.0, 1.0]] * 3)
+    gates = torch.tensor([[0.5, 0.9, 0.25]] * 3)
+    memory, out = torch.zeros(1, 1, D, Dv), torch.zeros(3, Dv)
+    k.gated_delta_scan(rows, gates, 1.0, batch, memory, out, 1, 1, D, Dv)
+    s, want = 0.0, []
+    for _ in range(3):
+        s = 0.5 * s + 0.25 * (5.0 - 0.5 * s)
+        want.append(s)
+    assert_close(out[:, 0], torch.tensor(want), 1e-6)
+
+
+def test_parallel_mixer_in_the_layers_own_product():
+    """Two sides with their scales, alone and as part of the layer's one product with the feed-forward; the residual multiplier;
+    a layer without feed-forward."""
+    from kvcache_b200.parts.base import ScaledDelta
+    from kvcache_b200.parts.block import ParallelBlock
+    from kvcache_b200.parts.feedforward import PlainMLP
+    from kvcache_b200.parts.norm import RMSNorm
+    from kvcache_b200.parts.recurrent import ParallelMixer
+    T, W, eps = 21, 20, 1e-5
+    left = dict(heads=4, kv_heads=2, dim=6, vdim=3, scale=1.1, mask={"size": 5, "keep_first": 2})
+    right = {"heads": 2, "kv_heads": 1, "dim": 5, "vdim": 7, "conv": 3}
+    m = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 1.6}
+
+    def make():
+        from kvcache_b200.parts.recurrent import GatedDeltaMixer
+        d = GatedDeltaMixer(W, 2, 1, 5, 7, 3, eps=eps, prefix="l0.mix.right.", dtype="float32", decay_rank=4, gate_rank=3)
+        return ParallelMixer(W, _attention_part(W, left, "g", prefix="l0.mix.left."), d, 0.7, 1.6, "float32")
+    mlp = PlainMLP(W, 13, activation="gelu", prefix="l0.mlp.", dtype="float32")
+    blocks = [ParallelBlock(W, RMSNorm(W, eps, "l0.norm1"), make(), ffn, "float32", gain=0.4) for ffn in (mlp, None)]
+    w = _weights(blocks[0].tensor_specs(), 8)
+    wd = {k: v.double() for k, v in w.items()}
+    x = torch.randn(T, W, generator=torch.Generator().manual_seed(9))
+    mixer = make()
+    mixer.bind(w, torch.device("cpu"))
+    batch, kv = _scenario([(0, T)], mixer.cache_spec(), slots=[1])
+    want = plain.mixer_forward("parallel", m, wd, "l0.mix.", x.double(), torch.arange(T), eps)
+    assert_close(mixer.forward(x, _context(batch, kv, _states(mixer))), want, 1e-5, "the mixer alone")
+    for block, ff in zip(blocks, ({"kind": "dense"}, None)):
+        block.bind(w, torch.device("cpu"))
+        config = {"layers": [{"type": "parallel", "mixer": m, "mlp": ff}], "norm": {"eps": eps}, "residual_mult": 0.4}
+        _, kv = _scenario([(0, T)], mixer.cache_spec(), slots=[1])
+        delta = block.forward(x.clone(), None, _context(batch, kv, _states(mixer)))
+        assert isinstance(delta, ScaledDelta)
+        assert_close(x.double() + delta.delta.double() * delta.scale.double(), plain.layer_forward(config, wd, 0, x.double(), torch.arange(T)), 1e-5)
+        assert block.weight_bytes() > 0
+    with pytest.raises(ValueError):
+        ParallelBlock(W, RMSNorm(W, eps, "n"), make(), object(), "float32")
+
+
+def test_exact_gelu_feed_forward():
+    from kvcache_b200.parts.feedforward import PlainMLP
+    T, W, F = 9, 20, 24
+    part = PlainMLP(W, F, activation="gelu", prefix="f.", dtype="float32")
+    w = _weights(part.tensor_specs(), 5, std=0.6)
+    part.bind(w, torch.device("cpu"))
+    x = torch.randn(T, W, generator=torch.Generator().manual_seed(6))
+    wd = {k: v.double() for k, v in w.items()}
+    want = plain.feed_forward(wd, "f.", x.double())
+    assert_close(part.forward(x, _context()), want, 1e-6)
+    z = x.double() @ wd["f.up"].t()
+    tanh_form = 0.5 * z * (1 + torch.tanh((2 / torch.pi) ** 0.5 * (z + 0.044715 * z ** 3)))
+    assert (tanh_form @ wd["f.down"].t() - want).abs().max() > 20 * 1e-6 * want.abs().max(), "the other gelu differs by more"
+    wide = torch.full((T, F + 7), 3.0)
+    part.forward_hidden(x, _context(), wide, 5)
+    assert_close(wide[:, 5:5 + F], plain.exact_gelu(z), 1e-6)
+    assert bool((wide[:, :5] == 3.0).all()) and bool((wide[:, 5 + F:] == 3.0).all())
+
+
+def test_residual_stream_after_every_layer_run(tmp_path):
+    """Run by run, the passes of the loop among them: a model cut after k layer runs (its final norm with weight 1, its head the
+    identity) gives the plain implementation's residual stream after run k, divided by its root mean square."""
+    from kvcache_b200.cache import CacheManager
+    from kvcache_b200.engine.loading import load_model
+    from kvcache_b200.engine.runner import ModelRunner, StepEntry
+    folder = make_kaposun_folder(tmp_path, "A")
+    config, weights = plain.read_folder(folder)
+    tokens = random_tokens(config["vocab"], 37, 3)
+    streams = []
+    plain.forward(config, weights, tokens, streams)
+    assert len(streams) == 5
+    for k in range(1, len(streams) + 1):
+        model = load_model(folder, "float32", "cpu", max_positions=64)
+        model.schedule = model.schedule[:k]
+        model._writers = {c.cache: c.layer for c in model.schedule}
+        model.final_norm.weight, model.final_norm.eps = torch.ones(model.width), 0.0
+        model.head, model.vocab_size = torch.eye(model.width), model.width
+        cache = CacheManager(model.cache_entries(), page_size=8, num_pages=16, max_slots=1, max_tokens_per_request=64, dtype="float32", device="cpu")
+        runner = ModelRunner(model, cache, TorchKernels(wide=True), max_tokens_per_step=64)
+        got = runner.step([StepEntry(cache.admit(), tokens, list(range(len(tokens))))])
+        assert_close(got, plain.rms_norm(streams[k - 1], torch.ones(model.width, dtype=torch.float64), 0.0), 1e-5, f"after run {k}")
+
+
+# ---- the model in the engine ------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_whole_prompt_and_its_first_tokens(tmp_path, name):
+    runner, config, weights = _runner(tmp_path, name)
+    tokens = random_tokens(config["vocab"], 75, 1)
+    want = plain.forward(config, weights, tokens)
+    assert_close(replay_modes.whole(runner, tokens), want, REL)
+    assert runner.cache.used_pages() == 0
+    for n in (1, 2, 3):
+        assert_close(replay_modes.whole(runner, tokens[:n]), want[:n], REL, f"first {n}")
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_prefill_against_token_by_token_decoding(tmp_path, name):
+    runner, config, weights = _runner(tmp_path, name)
+    tokens = random_tokens(config["vocab"], 60, 2)
+    want = plain.forward(config, weights, tokens)
+    assert_close(replay_modes.last_32_one_by_one(runner, tokens), want[-33:], REL)
+    assert_close(replay_modes.portions(runner, tokens, [1] * 60), want, REL, "every token alone")
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_portions_down_to_two_tokens(tmp_path, name):
+    runner, config, weights = _runner(tmp_path, name)
+    tokens = random_tokens(config["vocab"], 101, 3)
+    want = plain.forward(config, weights, tokens)
+    assert_close(replay_modes.portions(runner, tokens, [2, 17, 3, 31, 2, 16, 8, 22]), want, REL)
+    assert_close(replay_modes.portions(runner, tokens, [40, 2, 2, 5, 52]), want, REL)
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_mixed_batches_with_pages_and_slots_used_again(tmp_path, name):
+    """Unequal requests beside one another against each alone; a and b end and d and e take their pages and slots, which hold
+    other requests' keys, states and convolution inputs."""
+    runner, config, weights = _runner(tmp_path, name, num_pages=replay_modes.mixed_pool_tokens() // PAGE_SIZE[name])
+    seqs = {k: random_tokens(config["vocab"], n, 10 + i) for i, (k, n) in enumerate(replay_modes.MIXED_LENGTHS)}
+    got = replay_modes.mixed(runner, seqs)
+    for k, tokens in seqs.items():
+        assert_close(got[k], plain.forward(config, weights, tokens), REL, k)
+
+
+def _masks(config):
+    return [layer["mixer"]["left"]["mask"] for layer in config["layers"] if layer["type"] == "parallel" and "mask" in layer["mixer"]["left"]]
+
+
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_sharp_attention_at_the_edges_in_prompts_and_decoding(tmp_path, name):
+    """With the score scale multiplied the softmax of most heads rests on single keys: a window or a run of kept tokens one token
+    too long or too short changes the logits by far more than the tolerance."""
+    runner, config, weights = _runner(tmp_path, name, sharpen=12.0, max_tokens_per_step=256, max_tokens_per_request=256)
+    tokens = random_tokens(config["vocab"], 120, 5)
+    want = plain.forward(config, weights, tokens)
+    for key in ("size", "keep_first"):
+        for delta in (-1, 1):
+            other = copy.deepcopy(config)
+            for mask in _masks(other):
+                mask[key] = max(1 if key == "size" else 0, mask[key] + delta)
+            if other != config:
+                assert (plain.forward(other, weights, tokens) - want).abs().max() > 0.01 * want.abs().max(), (key, delta)
+    assert_close(replay_modes.portions(runner, tokens, [7, 2, 27, 64, 3, 17]), want, 1e-3)
+    assert_close(replay_modes.portions(runner, tokens, [80] + [1] * 40), want, 1e-3, "the window passes over decoded tokens")
+
+
+def test_positions_are_not_rotated_in_the_window_layers_and_are_in_the_others(tmp_path):
+    """A longer context in front of the same tokens: kept as a fact of the plain implementation, so that the engine's agreement
+    with it means something."""
+    config, weights = plain.read_folder(make_kaposun_folder(tmp_path, "A"))
+    bare = copy.deepcopy(config)
+    bare["layers"][1]["mixer"].pop("rot")
+    unscaled = copy.deepcopy(config)
+    unscaled["layers"][1]["mixer"]["rot"].pop("scaling")
+    tokens = random_tokens(config["vocab"], 40, 9)
+    want = plain.forward(config, weights, tokens)
+    for other in (bare, unscaled):
+        assert (plain.forward(other, weights, tokens) - want).abs().max() > 100 * REL * want.abs().max()
+
+
+def test_every_pass_of_a_loop_keeps_its_own_state(tmp_path):
+    """C's loop holds recurrent layers: three passes, three states per layer, none of them shared, all moved on by decoding."""
+    from kvcache_b200.engine.runner import StepEntry
+    runner, config, weights = _runner(tmp_path, "C")
+    tokens = random_tokens(config["vocab"], 30, 4)
+    slot = runner.cache.admit()
+    runner.step([StepEntry(slot, tokens[:29], [])])
+    out = runner.step([StepEntry(slot, tokens[29:], [0])]).clone()
+    assert_close(out, plain.forward(config, weights, tokens)[-1:], REL)
+    passes = [runner.cache.states[i]["right.memory"][slot] for i in (1, 3, 5)]
+    assert all((a - b).abs().max() > 1e-2 * a.abs().max() for a, b in zip(passes, passes[1:]))
+
+
+def test_long_decoding(tmp_path):
+    runner, config, weights = _runner(tmp_path, "A", max_tokens_per_step=512, max_tokens_per_request=512)
+    tokens = random_tokens(config["vocab"], 220, 6)
+    got = replay_modes.portions(runner, tokens, [20] + [1] * 200)
+    assert_close(got, plain.forward(config, weights, tokens), REL)
+
+
+def test_pages_behind_the_window_are_given_back_and_kept_ones_stay(tmp_path):
+    """C has only a windowed attention: a long request never holds more pages than its kept tokens, its window and a portion span."""
+    from kvcache_b200.engine.runner import StepEntry
+    runner, config, weights = _runner(tmp_path, "C", num_pages=24, max_tokens_per_step=64, max_tokens_per_request=512)
+    tokens = random_tokens(config["vocab"], 150, 8)
+    slot, at, most, got = runner.cache.admit(), 0, 0, []
+    for n in [16] * 5 + [1] * 70:
+        got.append(runner.step([StepEntry(slot, tokens[at:at + n], list(range(n)))]).clone())
+        at += n
+        most = max(most, runner.cache.used_pages())
+    assert_close(torch.cat(got), plain.forward(config, weights, tokens), REL)
+    assert most <= 3 + (5 - 1 + 16 + 3) // 4 + 1 and runner.cache.used_pages() <= 3 + 3
+    runner.cache.release(slot)
+    assert runner.cache.used_pages() == 0
+
+
+# ---- generation through the entry point and the scheduler -------------------------------------------------------------
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_greedy_generation_matches_plain(tmp_path, name):
+    from kvcache_b200 import LLM, SamplingParams
+    folder = make_kaposun_folder(tmp_path, name)
+    config, weights = plain.read_folder(folder)
+    prompts = [random_tokens(config["vocab"], n, 40 + n) for n in (1, 9, 24, 40)]
+    llm = LLM(folder, kernels=TorchKernels(), dtype="float32", device="cpu", page_size=PAGE_SIZE[name], num_pages=40, max_running=3,
+              max_tokens_per_step=48, chunk_size=16, use_graphs=False)
+    got = llm.generate(prompts, SamplingParams(max_new_tokens=6, ignore_eos=True))
+    for prompt, out in zip(prompts, got):
+        assert out == plain.greedy(config, weights, prompt, 6)
+    assert llm.core.cache.used_pages() == 0 and llm.last_stats.finished == len(prompts)
