@@ -47,7 +47,7 @@ struct ScanChunks {
     int L, S;              // tokens in a chunk; segments in the step
     float* local_S;        // [chunk, H, D, Dv]   end state of the chunk scanned from an empty state
     float* local_vec;      // [chunk, H, D]       channel decay: the product of the chunk's decays; exponential gates: its normaliser
-    float* local_F;        // [chunk, H]          exponential gates: the sum of the chunk's log forget gates; head decay: the product of its decays
+    float* local_F;        // [chunk, H]          exponential gates: the sum of the chunk's log forget gates
     float* local_m;        // [chunk, H]          exponential gates: the chunk's maximum from an empty state
     float* start_S;        // [chunk, H, D, Dv]   state before the chunk's first token
     float* start_vec;      // [chunk, H, D]       exponential gates: the normaliser there
@@ -179,7 +179,7 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
     for (int idx = threadIdx.x; idx < 2 * tile_floats; idx += blockDim.x) tile_s[idx] = 0.f;
     __syncthreads();
     if (n_rows > 0) stage(0, r0, min(TILE, n_rows));
-    float S[R], nz[NPL], total[NPL], total_keep = 1.f;
+    float S[R], nz[NPL], total[NPL];
     float* mem = memory + ((size_t)slot * H + h) * D * Dv;
     const size_t cid = (size_t)blockIdx.z * H + h;             // (chunk id, head) in the scratch arrays
     const bool from_slot = ch.start_S == nullptr;
@@ -260,7 +260,6 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
         if (MODE == SCAN_HEAD_DECAY) {
             keep = s_s[0];
             gain = s_s[TILE] * v;
-            if (PASS == SCAN_LOCAL) total_keep *= keep;
         } else if (MODE == SCAN_EXP_GATES) {
             keep = gate_s[0][tt];
             const float take = gate_s[1][tt];
@@ -371,7 +370,6 @@ __global__ void __launch_bounds__(512) matrix_state_scan_kernel(
     }
     if (blockIdx.x != 0 || warp != 0) return;
     if (MODE != SCAN_EXP_GATES) {
-        if (PASS == SCAN_LOCAL && MODE == SCAN_HEAD_DECAY && lane == 0) ch.local_F[cid] = total_keep;
         if (PASS == SCAN_LOCAL && MODE == SCAN_CHANNEL_DECAY)
 #pragma unroll
             for (int i = 0; i < NPL; ++i) {
@@ -429,8 +427,6 @@ __global__ void scan_chunk_starts_kernel(const int* __restrict__ seg_q_len, cons
             if (c + 1 == chunks) break;
             if (MODE == SCAN_CHANNEL_DECAY) {
                 s = ch.local_vec[cid * D + d] * s + ch.local_S[cid * per + e];
-            } else if (MODE == SCAN_HEAD_DECAY) {
-                s = ch.local_F[cid] * s + ch.local_S[cid * per + e];
             } else {
                 const float F = ch.local_F[cid], ml = ch.local_m[cid];
                 const float m1 = fmaxf(F + m, ml);
@@ -596,7 +592,9 @@ static int launch_scan(const float* proj, int P, int q_col, int k_col, int v_col
         KVB_SCAN_PASS(SCAN_FROM_START, S);
         return KVB_OK;
     }
-    if constexpr (scan_mixes_keys(MODE)) {
+    if constexpr (MODE == SCAN_HEAD_DECAY) {
+        return KVB_ERR_LIMIT;                                  // in one piece only
+    } else if constexpr (scan_mixes_keys(MODE)) {
         const int state_blocks = col_blocks;
         col_blocks = ((Dv + D + COLS - 1) / COLS + warps - 1) / warps;     // the transition's columns beside the state's
         KVB_SCAN_PASS(SCAN_LOCAL, max_chunks);
@@ -831,6 +829,61 @@ __device__ __forceinline__ float conv_channel(const ShortConv& cv, const ConvRow
     return acc / (1.f + expf(-acc));
 }
 
+// The same for a warp's CH x 32 channels c0 .. c0 + count - 1 and up to CONV_ROWS rows in turn, for convolutions of at most four
+// taps: weights are read once, inputs once per tile, and all of a tile's inputs are on their way together.  Same sums in the same
+// order.  `emit(r, y)` receives the warp's channels of row r.
+constexpr int CONV_ROWS = 8, CONV_TILE_TAPS = 4;
+template <int CH, typename Emit>
+__device__ __forceinline__ void conv_tile(const ShortConv& cv, int r0, int rows, int c0, int count, int lane, Emit emit) {
+    float w[CONV_TILE_TAPS][CH], bias[CH], before[CONV_TILE_TAPS - 1][CH], in[CONV_ROWS][CH];      // w[b], before[b - 1]: b tokens back
+#pragma unroll
+    for (int rr = 0; rr < CONV_ROWS; ++rr)
+#pragma unroll
+        for (int i = 0; i < CH; ++i)
+            in[rr][i] = rr < rows && lane + 32 * i < count ? cv.proj[(size_t)(r0 + rr) * cv.P + cv.col + c0 + lane + 32 * i] : 0.f;
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+        const int c = c0 + lane + 32 * i;
+        const bool ok = lane + 32 * i < count;
+        bias[i] = ok && cv.bias ? cv.bias[c] : 0.f;
+#pragma unroll
+        for (int b = 0; b < CONV_TILE_TAPS; ++b) w[b][i] = ok && b < cv.taps ? cv.w[(size_t)(cv.taps - 1 - b) * cv.C + c] : 0.f;
+    }
+    int seg_before = -1;
+#pragma unroll
+    for (int rr = 0; rr < CONV_ROWS; ++rr) {
+        if (rr >= rows) break;
+        const int r = r0 + rr, seg = cv.row_segment[r];
+        if (seg != seg_before) {                               // a tile's first row, or a segment's
+            const ConvRow cr = conv_row(cv, r);
+#pragma unroll
+            for (int b = 1; b < CONV_TILE_TAPS; ++b)
+#pragma unroll
+                for (int i = 0; i < CH; ++i) {
+                    const int c = c0 + lane + 32 * i;
+                    float x = 0.f;
+                    if (b < cv.taps && lane + 32 * i < count)
+                        x = b <= cr.t ? cr.row[c - (long long)b * cv.P] : cr.tail[(size_t)(cv.taps - 1 - b + cr.t) * cv.C + c];
+                    before[b - 1][i] = x;
+                }
+            seg_before = seg;
+        }
+        float y[CH];
+#pragma unroll
+        for (int i = 0; i < CH; ++i) {
+            float acc = bias[i];
+#pragma unroll
+            for (int b = CONV_TILE_TAPS - 1; b >= 1; --b) acc = fmaf(w[b][i], before[b - 1][i], acc);
+            acc = fmaf(w[0][i], in[rr][i], acc);
+            y[i] = acc / (1.f + expf(-acc));
+#pragma unroll
+            for (int b = CONV_TILE_TAPS - 1; b >= 2; --b) before[b - 1][i] = before[b - 2][i];
+            before[0][i] = in[rr][i];
+        }
+        emit(r, y);
+    }
+}
+
 // The state after the step: a thread per (segment, channel).  Entry j moves from entry j + rows of the old state or from the
 // segment's rows; going up, an entry is read before it is overwritten.
 __global__ void short_conv_tail_kernel(ShortConv cv, int S) {
@@ -860,7 +913,7 @@ __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1
 // gates[r] = [decays a = exp(-rate_h softplus(z + dt_bias)): H of D | write strengths sigmoid(proj[b_col + h]): H] (a head each).
 __global__ void gated_delta_inputs_kernel(ShortConv cv, int b_col, const float* __restrict__ z, int z_stride, const float* __restrict__ dt_bias,
                                           const float* __restrict__ rate, float unit_eps, float* __restrict__ rows,
-                                          float* __restrict__ gates, int total, int H, int G, int D, int Dv, int single) {
+                                          float* __restrict__ gates, int gate_stride, int total, int H, int G, int D, int Dv, int single) {
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31;
@@ -887,7 +940,7 @@ __global__ void gated_delta_inputs_kernel(ShortConv cv, int b_col, const float* 
         for (int d = lane; d < Dv; d += 32) out[c0 + d] = conv_channel(cv, cr, c0 + d, single);
     } else {
         const int h = job - 2 * G - H;
-        float* g = gates + (size_t)r * (H * D + H);
+        float* g = gates + (size_t)r * gate_stride;
         const float* zr = z + (size_t)r * z_stride + h * D;
         const float rt = rate[h];
         for (int d = lane; d < D; d += 32) g[h * D + d] = expf(-rt * softplus(zr[d] + dt_bias[h * D + d]));
@@ -895,32 +948,95 @@ __global__ void gated_delta_inputs_kernel(ShortConv cv, int b_col, const float* 
     }
 }
 
+// The same, a warp per (tile of CONV_ROWS rows, job): steps of many rows.  CH: 32nds of a head's channels (a v head's in runs).
+template <int CH>
+__global__ void __launch_bounds__(128) gated_delta_inputs_tile_kernel(ShortConv cv, int b_col, const float* __restrict__ z, int z_stride,
+                                                                      const float* __restrict__ dt_bias, const float* __restrict__ rate,
+                                                                      float unit_eps, float* __restrict__ rows, float* __restrict__ gates,
+                                                                      int gate_stride, int T, int total, int H, int G, int D, int Dv) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (id >= total) return;
+    const int v_runs = (H * Dv + 32 * CH - 1) / (32 * CH), jobs = 2 * G + v_runs + H;
+    const int tile = id / jobs, job = id - tile * jobs, r0 = tile * CONV_ROWS, n = min(CONV_ROWS, T - r0);
+    if (job < 2 * G) {
+        conv_tile<CH>(cv, r0, n, job * D, D, lane, [&](int r, const float (&y)[CH]) {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < CH; ++i) ss += lane + 32 * i < D ? y[i] * y[i] : 0.f;
+            const float inv = 1.f / sqrtf(warp_sum(ss) + unit_eps);
+#pragma unroll
+            for (int i = 0; i < CH; ++i)
+                if (lane + 32 * i < D) rows[(size_t)r * cv.C + job * D + lane + 32 * i] = y[i] * inv;
+        });
+    } else if (job < 2 * G + v_runs) {
+        const int first = (job - 2 * G) * 32 * CH, c0 = 2 * G * D + first, count = min(32 * CH, H * Dv - first);
+        conv_tile<CH>(cv, r0, n, c0, count, lane, [&](int r, const float (&y)[CH]) {
+#pragma unroll
+            for (int i = 0; i < CH; ++i)
+                if (lane + 32 * i < count) rows[(size_t)r * cv.C + c0 + lane + 32 * i] = y[i];
+        });
+    } else {
+        const int h = job - 2 * G - v_runs;
+        const float rt = rate[h];
+#pragma unroll
+        for (int i = 0; i < CH; ++i) {
+            const int d = lane + 32 * i;
+            if (d >= D) break;
+            const float bias = dt_bias[h * D + d];
+            float zr[CONV_ROWS];
+#pragma unroll
+            for (int rr = 0; rr < CONV_ROWS; ++rr) zr[rr] = rr < n ? z[(size_t)(r0 + rr) * z_stride + h * D + d] : 0.f;
+#pragma unroll
+            for (int rr = 0; rr < CONV_ROWS; ++rr)
+                if (rr < n) gates[(size_t)(r0 + rr) * gate_stride + h * D + d] = expf(-rt * softplus(zr[rr] + bias));
+        }
+        if (lane < n) gates[(size_t)(r0 + lane) * gate_stride + H * D + h] = 1.f / (1.f + expf(-cv.proj[(size_t)(r0 + lane) * cv.P + b_col + h]));
+    }
+}
+
+constexpr int CONV_TILE_MIN_ROWS = 128;      // steps of at least this many rows take the kernels with tiles of rows
+
 // proj: float32 [T, P] with the projections [q | k | v] at `col` and the write-strength logits at `b_col`; z: the decay logits
 // (columns 0 .. H * D of rows of z_stride); rate [H] = exp of the learned log rates; rows [T, 2 G D + H Dv] and gates
-// [T, H D + H] float32 are what kvb_gated_delta_scan reads.  `tail` moves on by the step's rows.
+// [T, gate_stride] float32 are what kvb_gated_delta_scan reads.  `tail` moves on by the step's rows.
 KVB_API int kvb_gated_delta_inputs(const float* proj, int P, int col, int b_col, const float* conv_w, int taps, float* tail, const float* z,
                                    int z_stride, const float* dt_bias, const float* rate, float unit_eps, float* rows, float* gates,
-                                   const int* row_segment, const int* seg_q_start, const int* seg_q_len, const int* seg_slot, int T, int S,
+                                   int gate_stride, const int* row_segment, const int* seg_q_start, const int* seg_q_len, const int* seg_slot, int T, int S,
                                    int H, int G, int D, int Dv, cudaStream_t stream) {
     if (T <= 0 || S <= 0) return KVB_OK;
-    if (H < 1 || G < 1 || H % G || D < 1 || Dv < 1 || taps < 1 || z_stride < H * D) return KVB_ERR_SHAPE;
+    if (H < 1 || G < 1 || H % G || D < 1 || Dv < 1 || taps < 1 || z_stride < H * D || gate_stride < H * D + H) return KVB_ERR_SHAPE;
     if (D > 256 || S > 65535 || (long long)T * (2 * G + 2 * H) > 0x7fffffffLL) return KVB_ERR_LIMIT;
     const ShortConv cv = {proj, P, col, 2 * G * D + H * Dv, taps, conv_w, nullptr, tail, row_segment, seg_q_start, seg_q_len, seg_slot};
+    if (T >= CONV_TILE_MIN_ROWS && T != S && taps <= CONV_TILE_TAPS) {
+        const int tiles = (T + CONV_ROWS - 1) / CONV_ROWS;
+#define KVB_DELTA_TILES(CH)                                                                                                         \
+    do {                                                                                                                            \
+        const int n = tiles * (2 * G + (H * Dv + 32 * CH - 1) / (32 * CH) + H);                                                     \
+        kvb_launch(gated_delta_inputs_tile_kernel<CH>, dim3((n + 3) / 4), dim3(128), 0, stream, cv, b_col, z, z_stride, dt_bias, rate, \
+                   unit_eps, rows, gates, gate_stride, T, n, H, G, D, Dv);                                                          \
+    } while (0)
+        if (D <= 64) KVB_DELTA_TILES(2); else if (D <= 128) KVB_DELTA_TILES(4); else KVB_DELTA_TILES(8);
+#undef KVB_DELTA_TILES
+        return launch_conv_tail(cv, T, S, stream);
+    }
     const int total = T * (2 * G + 2 * H), warps = 4;
     kvb_launch(gated_delta_inputs_kernel, dim3((total + warps - 1) / warps), dim3(32 * warps), 0, stream, cv, b_col, z, z_stride, dt_bias,
-               rate, unit_eps, rows, gates, total, H, G, D, Dv, T == S ? 1 : 0);
+               rate, unit_eps, rows, gates, gate_stride, total, H, G, D, Dv, T == S ? 1 : 0);
     return launch_conv_tail(cv, T, S, stream);
 }
 
 // The gated delta rule over the tokens of every segment, from and into memory[slot] ([H, D, Dv], float32); rows and gates as made
 // by kvb_gated_delta_inputs.  out = q_scale S'^T q.  `max_chunks` > 0: the chunked form, as for the other scans, with `scratch`
 // of max_chunks * H * (2 D Dv + D D + 2 D + 3) floats.
-KVB_API int kvb_gated_delta_scan(const float* rows, const float* gates, float q_scale, const int* seg_q_start, const int* seg_q_len,
+KVB_API int kvb_gated_delta_scan(const float* rows, const float* gates, int gate_stride, float q_scale, const int* seg_q_start, const int* seg_q_len,
                                  const int* seg_slot, float* memory, float* out, int T, int S, int H, int G, int D, int Dv, int chunk_len,
                                  int max_chunks, float* scratch, cudaStream_t stream) {
     if (S <= 0 || T <= 0) return KVB_OK;
-    if (G < 1 || H % G) return KVB_ERR_SHAPE;
-    return scan_any(SCAN_GATED_DELTA, rows, 2 * G * D + H * Dv, 0, G * D, 2 * G * D, gates, H * D + H, 0, H * D, 0.f, q_scale, 0.f, seg_q_start,
+    if (G < 1 || H % G || gate_stride < H * D + H) return KVB_ERR_SHAPE;
+    return scan_any(SCAN_GATED_DELTA, rows, 2 * G * D + H * Dv, 0, G * D, 2 * G * D, gates, gate_stride, 0, H * D, 0.f, q_scale, 0.f, seg_q_start,
                     seg_q_len, seg_slot, memory, nullptr, nullptr, out, T, S, H, D, Dv, chunk_len, max_chunks, scratch, stream, true, G);
 }
 
@@ -950,6 +1066,34 @@ __global__ void state_space_inputs_kernel(ShortConv cv, int dt_col, const float*
     }
 }
 
+// The same, a warp per (tile of CONV_ROWS rows, job).
+__global__ void __launch_bounds__(128) state_space_inputs_tile_kernel(ShortConv cv, int dt_col, const float* __restrict__ dt_bias,
+                                                                      const float* __restrict__ rate, float* __restrict__ rows,
+                                                                      float* __restrict__ gates, int T, int total, int H) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (id >= total) return;
+    const int jobs = (cv.C + CONV_RUN - 1) / CONV_RUN + 1, tile = id / jobs, job = id - tile * jobs;
+    const int r0 = tile * CONV_ROWS, n = min(CONV_ROWS, T - r0);
+    if (job + 1 < jobs) {
+        const int c0 = job * CONV_RUN, count = min(CONV_RUN, cv.C - c0);
+        conv_tile<CONV_RUN / 32>(cv, r0, n, c0, count, lane, [&](int r, const float (&y)[CONV_RUN / 32]) {
+#pragma unroll
+            for (int i = 0; i < CONV_RUN / 32; ++i)
+                if (lane + 32 * i < count) rows[(size_t)r * cv.C + c0 + lane + 32 * i] = y[i];
+        });
+    } else {
+        for (int i = lane; i < n * H; i += 32) {
+            const int r = r0 + i / H, h = i - i / H * H;
+            const float d = softplus(cv.proj[(size_t)r * cv.P + dt_col + h] + dt_bias[h]);
+            gates[(size_t)r * 2 * H + h] = expf(-rate[h] * d);
+            gates[(size_t)r * 2 * H + H + h] = d;
+        }
+    }
+}
+
 // proj: float32 [T, P] with the C convolved channels [x: H Dv | B: G N | C: G N] at `col` and the step sizes at `dt_col`; rows
 // [T, C] and gates [T, 2 H] float32 are what kvb_state_space_scan reads.  `tail` moves on by the step's rows.
 KVB_API int kvb_state_space_inputs(const float* proj, int P, int col, int C, int dt_col, const float* conv_w, const float* conv_b, int taps,
@@ -961,6 +1105,11 @@ KVB_API int kvb_state_space_inputs(const float* proj, int P, int col, int C, int
     const int jobs = (C + CONV_RUN - 1) / CONV_RUN + 1, warps = 4;
     if (S > 65535 || (long long)T * jobs > 0x7fffffffLL) return KVB_ERR_LIMIT;
     const ShortConv cv = {proj, P, col, C, taps, conv_w, conv_b, tail, row_segment, seg_q_start, seg_q_len, seg_slot};
+    if (T >= CONV_TILE_MIN_ROWS && T != S && taps <= CONV_TILE_TAPS) {
+        const int n = (T + CONV_ROWS - 1) / CONV_ROWS * jobs;
+        kvb_launch(state_space_inputs_tile_kernel, dim3((n + 3) / 4), dim3(128), 0, stream, cv, dt_col, dt_bias, rate, rows, gates, T, n, H);
+        return launch_conv_tail(cv, T, S, stream);
+    }
     const int total = T * jobs;
     kvb_launch(state_space_inputs_kernel, dim3((total + warps - 1) / warps), dim3(32 * warps), 0, stream, cv, dt_col, dt_bias, rate, rows,
                gates, total, H, T == S ? 1 : 0);
@@ -968,14 +1117,14 @@ KVB_API int kvb_state_space_inputs(const float* proj, int P, int col, int C, int
 }
 
 // S' = decay S + d B x^T, out = S'^T C over the tokens of every segment, from and into memory[slot] ([H, N, Dv], float32); head h
-// reads B and C of group h / (H / G); rows and gates as made by kvb_state_space_inputs.
+// reads B and C of group h / (H / G); rows and gates as made by kvb_state_space_inputs.  In one piece: the form for single tokens
+// and short portions (long ones: scan_wide.cu).
 KVB_API int kvb_state_space_scan(const float* rows, const float* gates, const int* seg_q_start, const int* seg_q_len, const int* seg_slot,
-                                 float* memory, float* out, int T, int S, int H, int G, int N, int Dv, int chunk_len, int max_chunks,
-                                 float* scratch, cudaStream_t stream) {
+                                 float* memory, float* out, int T, int S, int H, int G, int N, int Dv, cudaStream_t stream) {
     if (S <= 0 || T <= 0) return KVB_OK;
     if (G < 1 || H % G) return KVB_ERR_SHAPE;
     return scan_any(SCAN_HEAD_DECAY, rows, H * Dv + 2 * G * N, H * Dv + G * N, H * Dv, 0, gates, 2 * H, 0, H, 0.f, 1.f, 0.f, seg_q_start,
-                    seg_q_len, seg_slot, memory, nullptr, nullptr, out, T, S, H, N, Dv, chunk_len, max_chunks, scratch, stream, true, G);
+                    seg_q_len, seg_slot, memory, nullptr, nullptr, out, T, S, H, N, Dv, 0, 0, nullptr, stream, true, G);
 }
 
 // out[t, out_col + i] = y_i / sqrt(mean over i's part of y^2 + eps) * w_i * scale with y_i = (o[t, i] + skip[i / Dv] x[t, i]) silu(g[t, i]);

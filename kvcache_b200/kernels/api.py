@@ -119,20 +119,26 @@ _SIGNATURES = {
         "kvb_head_gate": [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_int,
                           _c_int, _c_void_p],
         "kvb_gated_delta_inputs": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
-                                   _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
-                                   _c_int, _c_int, _c_int, _c_void_p],
-        "kvb_gated_delta_scan": [_c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
-                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+                                   _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                                   _c_int, _c_int, _c_int, _c_int, _c_void_p],
+        "kvb_gated_delta_scan": [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
+                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+        "kvb_state_space_scan": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
+                                 _c_int, _c_int, _c_int, _c_void_p],
         "kvb_state_space_inputs": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
                                    _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
-        "kvb_state_space_scan": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
-                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
         "kvb_gate_part_norm": [_c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_float, _c_float,
                                _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_lightning_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                                _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
         "kvb_bigram_embed": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                              _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    },
+    "scan_wide": {
+        "kvb_gated_delta_scan_wide": [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
+                                      _c_int, _c_int, _c_int, _c_int, _c_void_p],
+        "kvb_state_space_scan_wide": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
+                                      _c_int, _c_int, _c_void_p],
     },
     "attention_generic": {
         "kvb_paged_attention_kv": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
@@ -289,6 +295,7 @@ class CudaKernels(KernelSet):
         self._gemm_simt = _Library("gemm_simt")
         self._latent = _Library("latent")
         self._recurrent = _Library("recurrent")
+        self._scan_wide = _Library("scan_wide")
         self._moe = _Library("moe")
         self._latent_flash = _Library("latent_flash")
         self._gemm_grouped = _Library("gemm_grouped")
@@ -1359,15 +1366,6 @@ class CudaKernels(KernelSet):
             _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out), T, batch.num_segments,
             H, D, chunk, max_chunks, _ptr(scratch), self._stream()), "delta_rule_scan")
 
-    def _chunks(self, batch: StepBatch, workspace, floats_per_chunk: int, chunk: int):
-        """(chunk bound, scratch) of a scan in chunks of `chunk` tokens, or (0, None) where segments are scanned in one piece.
-        Sized by the step's rows and segments alone, so that a recorded step finds the same launches."""
-        if not self.SCAN_CHUNK or batch.max_q_len < self.SCAN_CHUNK_MIN_ROWS:
-            return 0, None
-        self.launches += 2
-        bound = -(-batch.num_tokens // chunk) + batch.num_segments
-        return bound, workspace.buffer("recurrent.mixing_chunks", (bound * floats_per_chunk,), torch.float32)
-
     def _conv_launches(self, batch: StepBatch, taps: int) -> None:
         self.launches += 1 if batch.num_tokens != batch.num_segments and taps > 1 else 0     # the state's own launch
 
@@ -1381,18 +1379,24 @@ class CudaKernels(KernelSet):
                            gates: torch.Tensor, H: int, G: int, D: int, Dv: int) -> None:
         """rows = silu of the causal convolution (weights `conv_w` [taps, channels]) of columns [q: G D | k: G D | v: H Dv] of
         `proj`, q and k divided by sqrt(sum of squares + unit_eps) per head; gates = [exp(-rate_h softplus(z + dt_bias)): H D |
-        sigmoid(proj[:, b_col + h]): H].  `tail` [slots, taps - 1, channels]: the request's last inputs, moved on."""
+        sigmoid(proj[:, b_col + h]): H] (and columns after them that nobody reads).  `tail` [slots, taps - 1, channels]: the request's last inputs, moved on."""
         self._float32_only("gated_delta_inputs", proj, conv_w, tail, z, dt_bias, rate, rows, gates)
         T, C, taps = proj.shape[0], 2 * G * D + H * Dv, conv_w.shape[0]
         if (tuple(conv_w.shape) != (taps, C) or tuple(tail.shape[1:]) != (taps - 1, C) or tuple(rows.shape) != (T, C)
-                or tuple(gates.shape) != (T, H * D + H) or dt_bias.numel() != H * D or rate.numel() != H or b_col < C):
+                or gates.shape[0] != T or gates.shape[1] < H * D + H or dt_bias.numel() != H * D or rate.numel() != H or b_col < C):
             raise KernelError("gated_delta_inputs: the sizes do not fit one another")
         self._count("gated_delta_inputs")
         self._conv_launches(batch, taps)
         _check(self._recurrent.kvb_gated_delta_inputs(
             _ptr(proj), proj.shape[1], 0, b_col, _ptr(conv_w), taps, _ptr(tail), _ptr(z), z.shape[1], _ptr(dt_bias), _ptr(rate),
-            float(unit_eps), _ptr(rows), _ptr(gates), _ptr(batch.row_segment), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len),
+            float(unit_eps), _ptr(rows), _ptr(gates), gates.shape[1], _ptr(batch.row_segment), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len),
             _ptr(batch.seg_slot), T, batch.num_segments, H, G, D, Dv, self._stream()), "gated_delta_inputs")
+
+    # Portions of at least this many rows go through the scan that spreads a column over many lanes (csrc/scan_wide.cu): the state
+    # space always, the gated delta rule where a head has more key channels than DELTA_WIDE_ABOVE - with fewer, chunks that run side
+    # by side are ahead (2,048 rows, 14 heads of 64: 313 us in chunks, 478 us; 16 heads of 128: 810 us in chunks, 462 us).
+    SCAN_WIDE_MIN_ROWS = 64
+    DELTA_WIDE_ABOVE = 64
 
     def gated_delta_scan(self, rows: torch.Tensor, gates: torch.Tensor, q_scale: float, batch: StepBatch, memory: torch.Tensor,
                          out: torch.Tensor, H: int, G: int, D: int, Dv: int, workspace) -> None:
@@ -1401,12 +1405,22 @@ class CudaKernels(KernelSet):
         self._float32_only("gated_delta_scan", rows, gates, memory, out)
         if tuple(memory.shape[1:]) != (H, D, Dv):
             raise KernelError(f"the gated delta scan wants states [slots, {H}, {D}, {Dv}], got {tuple(memory.shape)}")
-        chunk = self.SCAN_CHUNK if batch.max_q_len < self.DELTA_LONG_ROWS else max(self.SCAN_CHUNK, self.DELTA_LONG_CHUNK)
-        max_chunks, scratch = self._chunks(batch, workspace, H * (2 * D * Dv + D * D + 2 * D + 3), chunk)
+        segments = (_ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out))
         self._count("gated_delta_scan")
-        _check(self._recurrent.kvb_gated_delta_scan(
-            _ptr(rows), _ptr(gates), float(q_scale), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory),
-            _ptr(out), rows.shape[0], batch.num_segments, H, G, D, Dv, chunk, max_chunks, _ptr(scratch), self._stream()), "gated_delta_scan")
+        if D > self.DELTA_WIDE_ABOVE and batch.max_q_len >= self.SCAN_WIDE_MIN_ROWS:
+            _check(self._scan_wide.kvb_gated_delta_scan_wide(_ptr(rows), _ptr(gates), gates.shape[1], float(q_scale), *segments,
+                                                             batch.num_segments, H, G, D, Dv, self._stream()), "gated_delta_scan (wide)")
+            return
+        max_chunks, scratch, chunk = 0, None, self.SCAN_CHUNK
+        if chunk and batch.max_q_len >= self.SCAN_CHUNK_MIN_ROWS:
+            if batch.max_q_len >= self.DELTA_LONG_ROWS:
+                chunk = max(chunk, self.DELTA_LONG_CHUNK)
+            max_chunks = -(-batch.num_tokens // chunk) + batch.num_segments          # as in `delta_rule_scan`
+            scratch = workspace.buffer("recurrent.delta_chunks", (max_chunks * H * (2 * D * Dv + D * D + 2 * D + 3),), torch.float32)
+            self.launches += 2
+        _check(self._recurrent.kvb_gated_delta_scan(_ptr(rows), _ptr(gates), gates.shape[1], float(q_scale), *segments, rows.shape[0],
+                                                    batch.num_segments, H, G, D, Dv, chunk, max_chunks, _ptr(scratch), self._stream()),
+               "gated_delta_scan")
 
     def state_space_inputs(self, proj: torch.Tensor, col: int, dt_col: int, conv_w: torch.Tensor, conv_b: torch.Tensor, tail: torch.Tensor,
                            dt_bias: torch.Tensor, rate: torch.Tensor, batch: StepBatch, rows: torch.Tensor, gates: torch.Tensor,
@@ -1426,17 +1440,20 @@ class CudaKernels(KernelSet):
             batch.num_segments, H, self._stream()), "state_space_inputs")
 
     def state_space_scan(self, rows: torch.Tensor, gates: torch.Tensor, batch: StepBatch, memory: torch.Tensor, out: torch.Tensor, H: int,
-                         G: int, N: int, Dv: int, workspace) -> None:
+                         G: int, N: int, Dv: int) -> None:
         """Per segment, from and into memory[slot] ([H, N, Dv], float32): S = decay S + d B x^T, out = S^T C; `rows` =
         [x: H Dv | B: G N | C: G N] and `gates` = [decay: H | d: H] as `state_space_inputs` makes them (head h: group h // (H / G))."""
         self._float32_only("state_space_scan", rows, gates, memory, out)
         if tuple(memory.shape[1:]) != (H, N, Dv) or rows.shape[1] != H * Dv + 2 * G * N:
             raise KernelError(f"the state-space scan wants states [slots, {H}, {N}, {Dv}], got {tuple(memory.shape)}")
-        max_chunks, scratch = self._chunks(batch, workspace, H * (2 * N * Dv + 2 * N + 3), self.SCAN_CHUNK)
+        segments = (_ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out))
         self._count("state_space_scan")
-        _check(self._recurrent.kvb_state_space_scan(
-            _ptr(rows), _ptr(gates), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out),
-            rows.shape[0], batch.num_segments, H, G, N, Dv, self.SCAN_CHUNK, max_chunks, _ptr(scratch), self._stream()), "state_space_scan")
+        if batch.max_q_len >= self.SCAN_WIDE_MIN_ROWS:
+            _check(self._scan_wide.kvb_state_space_scan_wide(_ptr(rows), _ptr(gates), *segments, batch.num_segments, H, G, N, Dv,
+                                                             self._stream()), "state_space_scan (wide)")
+        else:
+            _check(self._recurrent.kvb_state_space_scan(_ptr(rows), _ptr(gates), *segments, rows.shape[0], batch.num_segments, H, G, N, Dv,
+                                                        self._stream()), "state_space_scan")
 
     def gate_part_norm(self, o: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, gate, weight: torch.Tensor, eps: float, scale: float,
                        out: torch.Tensor, out_col: int, num_heads: int, value_dim: int, parts: int) -> None:

@@ -358,7 +358,7 @@ class GatedDeltaMixer(Mixer):
         z = ws.buffer("recurrent.z", (T, self.decay_size + self.heads_width), torch.float32)      # [decay logits | gate logits]
         k.linear(low, self.w_high, z)
         rows = ws.buffer("recurrent.rows", (T, self.channels), torch.float32)
-        gates = ws.buffer("recurrent.gates", (T, self.decay_size + H), torch.float32)
+        gates = ws.buffer("recurrent.gates", (T, self.decay_size + (H + 3) // 4 * 4), torch.float32)      # rows start on 16 bytes
         k.gated_delta_inputs(proj, self.channels, self.conv_w, ctx.state["conv"], z, self.dt_bias, self.rate, self.UNIT_EPS, ctx.batch,
                              rows, gates, H, G, D, V)
         o = ws.buffer("recurrent.o", (T, self.heads_width), torch.float32)
@@ -434,7 +434,7 @@ class StateSpaceMixer(Mixer):
         k.state_space_inputs(proj, W, W + self.channels, self.conv_w, self.conv_b, ctx.state["conv"], self.dt_bias, self.rate, ctx.batch,
                              rows, gates, H)
         y = ws.buffer("recurrent.o", (T, W), torch.float32)
-        k.state_space_scan(rows, gates, ctx.batch, ctx.state["memory"], y, H, self.groups, self.state, self.vdim, ws)
+        k.state_space_scan(rows, gates, ctx.batch, ctx.state["memory"], y, H, self.groups, self.state, self.vdim)
         k.gate_part_norm(y, rows, self.skip, (proj, 0), self.norm, self.eps, scale, out, out_col, H, self.vdim, self.norm_parts)
 
     def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:

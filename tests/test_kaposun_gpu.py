@@ -98,6 +98,7 @@ def test_head_gate_per_head_and_per_channel(kernels, dtype, per_channel, H, Dv, 
 
 
 SEGMENTS, SLOTS = [(0, 19), (50, 1), (7, 6), (3, 1), (9, 2)], [2, 0, 3, 5, 1]
+LONG_SEGMENTS, LONG_SLOTS = [(0, 101), (9, 1), (4, 2), (30, 1), (3, 50)], [1, 3, 0, 2, 5]      # tiles of rows that hold several segments
 SINGLES, SINGLE_SLOTS = [(4, 1), (0, 1), (77, 1)], [3, 1, 4]
 
 
@@ -112,8 +113,8 @@ def _to(case, device):
     return {k: v.clone().to(device) for k, v in case.items()}
 
 
-@pytest.mark.parametrize("H,G,D,Dv,taps", [(4, 2, 8, 12, 4), (3, 3, 33, 5, 2), (6, 1, 64, 64, 1), (2, 2, 128, 48, 5), (1, 1, 256, 16, 3), (16, 16, 64, 64, 4)])
-@pytest.mark.parametrize("segments,slots", [(SEGMENTS, SLOTS), (SINGLES, SINGLE_SLOTS)])
+@pytest.mark.parametrize("H,G,D,Dv,taps", [(4, 2, 8, 12, 4), (3, 3, 33, 5, 2), (6, 1, 64, 64, 1), (2, 2, 128, 48, 5), (1, 1, 256, 16, 3), (2, 1, 200, 130, 4), (16, 16, 64, 64, 4)])
+@pytest.mark.parametrize("segments,slots", [(SEGMENTS, SLOTS), (SINGLES, SINGLE_SLOTS), (LONG_SEGMENTS, LONG_SLOTS)])
 def test_gated_delta_inputs(kernels, H, G, D, Dv, taps, segments, slots):
     """Convolutions over portions (shorter and longer than the taps) and single tokens, unit queries and keys, decays, write
     strengths; the convolutions' state afterwards, other slots untouched."""
@@ -134,7 +135,7 @@ def test_gated_delta_inputs(kernels, H, G, D, Dv, taps, segments, slots):
 
 
 @pytest.mark.parametrize("H,C,taps,col", [(4, 100, 4, 7), (3, 128, 1, 0), (30, 300, 2, 64), (2, 17, 6, 3)])
-@pytest.mark.parametrize("segments,slots", [(SEGMENTS, SLOTS), (SINGLES, SINGLE_SLOTS)])
+@pytest.mark.parametrize("segments,slots", [(SEGMENTS, SLOTS), (SINGLES, SINGLE_SLOTS), (LONG_SEGMENTS, LONG_SLOTS)])
 def test_state_space_inputs(kernels, H, C, taps, col, segments, slots):
     batch = _segments_batch(segments, slots)
     T = batch.num_tokens
@@ -166,12 +167,13 @@ def _space_rows(T, H, G, N, Dv, seed=1):
     return _rand(T, H * Dv + 2 * G * N, seed=seed), gates
 
 
-def _run_scan(k, kind, rows, gates, batch, memory, sizes, ws):
+def _run_scan(k, kind, rows, gates, batch, memory, sizes):
+    from kvcache_b200.engine.workspace import Workspace
     out = torch.zeros(rows.shape[0], sizes[0] * sizes[3], device=rows.device)
     if kind == "delta":
-        k.gated_delta_scan(rows, gates, 0.3, batch, memory, out, *sizes, ws)
+        k.gated_delta_scan(rows, gates, 0.3, batch, memory, out, *sizes, Workspace(out.device))
     else:
-        k.state_space_scan(rows, gates, batch, memory, out, *sizes, ws)
+        k.state_space_scan(rows, gates, batch, memory, out, *sizes)
     return out
 
 
@@ -180,15 +182,14 @@ def _run_scan(k, kind, rows, gates, batch, memory, sizes, ws):
 def test_scans(kernels, kind, H, G, D, Dv):
     """Prompts, portions that continue a state, single tokens, states of other slots untouched; then every row alone, which must
     give the same bits as the rows together."""
-    from kvcache_b200.engine.workspace import Workspace
     batch = _segments_batch(SEGMENTS, SLOTS)
     T = batch.num_tokens
     rows, gates = (_delta_rows if kind == "delta" else _space_rows)(T, H, G, D, Dv)
     memory = _rand(6, H, D, Dv, seed=3)
     ref_mem, got_mem, one_mem = memory.clone(), memory.clone().to(DEV), memory.clone().to(DEV)
-    sizes, ws = (H, G, D, Dv), Workspace(DEV)
-    want = _run_scan(TorchKernels(wide=True), kind, rows, gates, batch, ref_mem, sizes, None)
-    got = _run_scan(kernels, kind, rows.to(DEV), gates.to(DEV), batch_to(batch, DEV), got_mem, sizes, ws)
+    sizes = (H, G, D, Dv)
+    want = _run_scan(TorchKernels(wide=True), kind, rows, gates, batch, ref_mem, sizes)
+    got = _run_scan(kernels, kind, rows.to(DEV), gates.to(DEV), batch_to(batch, DEV), got_mem, sizes)
     assert_close(got, want, 2e-5, "read-out")
     assert_close(got_mem, ref_mem, 2e-5, "states")
     assert torch.equal(got_mem[4].cpu(), memory[4])
@@ -196,43 +197,69 @@ def test_scans(kernels, kind, H, G, D, Dv):
     for (start, n), slot in zip(SEGMENTS, SLOTS):
         for i in range(n):
             single = batch_to(_segments_batch([(start + i, 1)], [slot]), DEV)
-            one = _run_scan(kernels, kind, rows[at:at + 1].to(DEV), gates[at:at + 1].to(DEV), single, one_mem, sizes, ws)
+            one = _run_scan(kernels, kind, rows[at:at + 1].to(DEV), gates[at:at + 1].to(DEV), single, one_mem, sizes)
             assert torch.equal(one, got[at:at + 1])
             at += 1
     assert torch.equal(one_mem, got_mem)
 
 
 @pytest.mark.parametrize("kind", ["delta", "space"])
-@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 64, 64), (1, 1, 33, 40), (2, 1, 128, 64), (3, 3, 8, 12), (2, 2, 200, 48), (2, 2, 128, 128)])
+@pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 64, 64), (1, 1, 33, 40), (2, 1, 128, 64), (3, 3, 8, 12), (2, 2, 200, 48), (2, 2, 128, 128), (2, 1, 100, 45),
+                                       (3, 1, 70, 5), (1, 1, 256, 33)])
 def test_scans_of_long_portions(kernels, kind, H, G, D, Dv):
-    """Portions long enough to be cut into chunks that run side by side: from an empty state and from a filled one, lengths that
-    are no multiple of the chunk, beside single tokens and short portions; against the plain recurrence."""
-    from kvcache_b200.engine.workspace import Workspace
+    """Portions for the scan that spreads a column over many lanes and for the one in chunks: many tiles of tokens, from an empty
+    state and from a filled one, lengths that are no multiple of a tile or a group, beside single tokens and short portions;
+    against the plain recurrence, and every segment alone, which must give the same bits (in the forms without chunks)."""
     segments, slots = [(0, 300), (50, 1), (100, 257), (3, 1), (0, 64), (5, 2)], [2, 0, 3, 5, 1, 4]
     batch = _segments_batch(segments, slots)
-    assert batch.max_q_len >= kernels.SCAN_CHUNK_MIN_ROWS
     T = batch.num_tokens
     rows, gates = (_delta_rows if kind == "delta" else _space_rows)(T, H, G, D, Dv)
     memory = _rand(7, H, D, Dv, seed=3)
     memory[2].zero_()
     ref_mem, got_mem = memory.clone(), memory.clone().to(DEV)
     sizes = (H, G, D, Dv)
-    want = _run_scan(TorchKernels(wide=True), kind, rows, gates, batch, ref_mem, sizes, None)
-    got = _run_scan(kernels, kind, rows.to(DEV), gates.to(DEV), batch_to(batch, DEV), got_mem, sizes, Workspace(DEV))
+    want = _run_scan(TorchKernels(wide=True), kind, rows, gates, batch, ref_mem, sizes)
+    got = _run_scan(kernels, kind, rows.to(DEV), gates.to(DEV), batch_to(batch, DEV), got_mem, sizes)
     kernels.check_errors()
     assert_close(got, want, 1e-4, "read-out")
     assert_close(got_mem, ref_mem, 1e-4, "states")
     assert torch.equal(got_mem[6].cpu(), memory[6])
+    if kind == "space" or D > kernels.DELTA_WIDE_ABOVE:
+        at, alone_mem = 0, memory.clone().to(DEV)
+        for (start, n), slot in zip(segments, slots):
+            if n >= kernels.SCAN_WIDE_MIN_ROWS:
+                alone = batch_to(_segments_batch([(start, n)], [slot]), DEV)
+                assert torch.equal(_run_scan(kernels, kind, rows[at:at + n].to(DEV), gates[at:at + n].to(DEV), alone, alone_mem, sizes), got[at:at + n])
+                assert torch.equal(alone_mem[slot], got_mem[slot])
+            at += n
+
+
+@pytest.mark.parametrize("D", [64, 96])
+def test_forms_of_the_delta_scan_agree(kernels, D):
+    """In one piece, in chunks, spread over lanes: the same read-outs and states up to rounding."""
+    H, G, Dv = 2, 1, 40
+    segments = [(0, 300), (4, 70)]
+    rows, gates = (t.to(DEV) for t in _delta_rows(370, H, G, D, Dv))
+    batch = batch_to(_segments_batch(segments, [1, 0]), DEV)
+    saved, results = (kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK), []
+    try:
+        for above, chunk in ((0, 64), (256, 64), (256, 0)):
+            kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK = above, chunk
+            memory = _rand(2, H, D, Dv, seed=3).to(DEV)
+            results.append((_run_scan(kernels, "delta", rows, gates, batch, memory, (H, G, D, Dv)), memory))
+    finally:
+        kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK = saved
+    for out, memory in results[1:]:
+        assert_close(out, results[0][0], 1e-5)
+        assert_close(memory, results[0][1], 1e-5)
 
 
 @pytest.mark.parametrize("kind", ["delta", "space"])
 @pytest.mark.parametrize("fast", [False, True])
 def test_scans_of_a_very_long_portion_with_slow_and_with_fast_decays(kernels, kind, fast):
-    """A portion long enough for the longer chunks; decays that hardly forget (early tokens reach the last read-outs) and decays
-    that underflow within a few tokens."""
-    from kvcache_b200.engine.workspace import Workspace
+    """Decays that hardly forget (early tokens reach the last read-outs) and decays that underflow within a few tokens."""
     H, G, D, Dv = 2, 2, 64, 64
-    segments, slots = [(10, kernels.DELTA_LONG_ROWS + 77), (0, 130), (5, 1)], [1, 0, 2]
+    segments, slots = [(10, 1613), (0, 130), (5, 1)], [1, 0, 2]
     batch = _segments_batch(segments, slots)
     T = batch.num_tokens
     rows, gates = (_delta_rows if kind == "delta" else _space_rows)(T, H, G, D, Dv)
@@ -240,8 +267,8 @@ def test_scans_of_a_very_long_portion_with_slow_and_with_fast_decays(kernels, ki
     keep.copy_(keep ** (150.0 if fast else 0.01))
     memory = _rand(3, H, D, Dv, seed=3)
     ref_mem, got_mem = memory.clone(), memory.clone().to(DEV)
-    want = _run_scan(TorchKernels(wide=True), kind, rows, gates, batch, ref_mem, (H, G, D, Dv), None)
-    got = _run_scan(kernels, kind, rows.to(DEV), gates.to(DEV), batch_to(batch, DEV), got_mem, (H, G, D, Dv), Workspace(DEV))
+    want = _run_scan(TorchKernels(wide=True), kind, rows, gates, batch, ref_mem, (H, G, D, Dv))
+    got = _run_scan(kernels, kind, rows.to(DEV), gates.to(DEV), batch_to(batch, DEV), got_mem, (H, G, D, Dv))
     kernels.check_errors()
     assert_close(got, want, 2e-4, "read-out")
     assert_close(got_mem, ref_mem, 2e-4, "states")
@@ -261,15 +288,14 @@ def test_gate_part_norm(kernels, dtype, H, Dv, parts, x_wide, g_col, wide, at):
 
 
 def test_sizes_that_do_not_fit_are_refused(kernels):
-    from kvcache_b200.engine.workspace import Workspace
     from kvcache_b200.kernels.api import KernelError
     batch = batch_to(_segments_batch([(0, 2)], [0]), DEV)
     rows, gates = (t.to(DEV) for t in _delta_rows(2, 2, 1, 8, 8))
-    out, ws = torch.zeros(2, 16, device=DEV), Workspace(DEV)
+    out = torch.zeros(2, 16, device=DEV)
     with pytest.raises(KernelError):
-        kernels.gated_delta_scan(rows, gates, 1.0, batch, torch.zeros(1, 2, 8, 9, device=DEV), out, 2, 1, 8, 8, ws)
+        kernels.gated_delta_scan(rows, gates, 1.0, batch, torch.zeros(1, 2, 8, 9, device=DEV), out, 2, 1, 8, 8, None)
     with pytest.raises(KernelError):
-        kernels.gated_delta_scan(rows, gates.double(), 1.0, batch, torch.zeros(1, 2, 8, 8, device=DEV), out, 2, 1, 8, 8, ws)
+        kernels.gated_delta_scan(rows, gates.double(), 1.0, batch, torch.zeros(1, 2, 8, 8, device=DEV), out, 2, 1, 8, 8, None)
     with pytest.raises(KernelError):
         kernels.gate_part_norm(out, out, torch.zeros(2, device=DEV), (out, 0), torch.ones(16, device=DEV), 1e-5, 1.0, out.clone(), 0, 2, 8, 3)
 
@@ -335,7 +361,7 @@ def test_four_ways_of_cutting(tmp_path, kernels, name, dtype):
 
 @pytest.mark.parametrize("name", ["A", "B", "C"])
 def test_float32_rows_do_not_depend_on_the_batch_or_the_cut(tmp_path, kernels, name):
-    """In float32 a position's logits are bit for bit the same alone, beside other requests, and in portions."""
+    """In float32 a position's logits are bit for bit the same alone, beside other requests, and in (short) portions."""
     runner, config, _ = _runner(tmp_path, kernels, name, "float32")
     from kvcache_b200.engine.runner import StepEntry
     a, b = random_tokens(config["vocab"], 40, 1), random_tokens(config["vocab"], 23, 2)

@@ -507,7 +507,7 @@ class TorchKernels:
         rows.copy_(torch.cat([qk.reshape(T, -1), y[:, 2 * G * D:]], dim=1).to(rows.dtype))
         soft = torch.nn.functional.softplus(z[:, :H * D].to(f) + dt_bias.to(f), threshold=1e9).view(T, H, D)
         decay = torch.exp(-rate.to(f)[None, :, None] * soft)
-        gates.copy_(torch.cat([decay.reshape(T, -1), torch.sigmoid(proj[:, b_col:b_col + H].to(f))], dim=1).to(gates.dtype))
+        gates[:, :H * D + H] = torch.cat([decay.reshape(T, -1), torch.sigmoid(proj[:, b_col:b_col + H].to(f))], dim=1).to(gates.dtype)
 
     def gated_delta_scan(self, rows, gates, q_scale, batch, memory, out, H, G, D, Dv, workspace=None):
         f = self.f
@@ -518,7 +518,7 @@ class TorchKernels:
                 q, k = (rows[t, c:c + G * D].to(f).view(G, D)[shared] for c in (0, G * D))
                 v = rows[t, 2 * G * D:].to(f).view(H, Dv)
                 S = gates[t, :H * D].to(f).view(H, D)[:, :, None] * S
-                u = gates[t, H * D:].to(f)[:, None] * (v - torch.einsum("hkv,hk->hv", S, k))
+                u = gates[t, H * D:H * D + H].to(f)[:, None] * (v - torch.einsum("hkv,hk->hv", S, k))
                 S = S + k[:, :, None] * u[:, None, :]
                 out[t] = (q_scale * torch.einsum("hkv,hk->hv", S, q)).reshape(-1).to(out.dtype)
             memory[slot] = S.to(memory.dtype)
@@ -529,7 +529,7 @@ class TorchKernels:
         d = torch.nn.functional.softplus(proj[:, dt_col:dt_col + H].to(f) + dt_bias.to(f), threshold=1e9)
         gates.copy_(torch.cat([torch.exp(-rate.to(f) * d), d], dim=1).to(gates.dtype))
 
-    def state_space_scan(self, rows, gates, batch, memory, out, H, G, N, Dv, workspace=None):
+    def state_space_scan(self, rows, gates, batch, memory, out, H, G, N, Dv):
         f = self.f
         shared = torch.arange(H) // (H // G)
         for lo, n, slot in self._segments(batch):
