@@ -45,6 +45,15 @@ __device__ __forceinline__ float gated_pair(float g, float u, float limit) {
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
 }
 
+// Activations of one number.  kind 0: tanh, 1: relu(v)^2, 2: cap * tanh(v / cap), 3: v Phi(v) with the normal distribution
+// function (the exact gelu).
+__device__ __forceinline__ float unary_activation(float v, int kind, float cap) {
+    if (kind == 0) return tanhf(v);
+    if (kind == 1) { const float p = fmaxf(v, 0.f); return p * p; }
+    if (kind == 2) return cap * tanhf(v / cap);
+    return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+}
+
 // Which keys up to its own a query at position `pos` sees, as one number `reach` (the `window` argument of the attention
 // kernels): w > 0 - the last w, so the first is max(0, pos - w + 1); -c < 0 - those of its chunk of c tokens, counted from the
 // request's first, so the first is pos - pos % c; 0 - all.  Returns the first.  It never decreases from one position to the next.

@@ -512,13 +512,6 @@ KVB_API int kvb_token_shift(int dtype, const void* x, const float* w, float* pre
 // out[t, out_col + i] = act(x[t, i]); kind 0: tanh, 1: relu(x)^2, 2: cap * tanh(x / cap), 3: x Phi(x) with the normal distribution
 // function (the exact gelu).  x: rows of x_stride, `cols` of them taken from x_col on; out may be x itself.  A thread takes VEC
 // neighbouring numbers of a row.
-__device__ __forceinline__ float activate(float v, int kind, float cap) {
-    if (kind == 0) return tanhf(v);
-    if (kind == 1) { const float p = fmaxf(v, 0.f); return p * p; }
-    if (kind == 2) return cap * tanhf(v / cap);
-    return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
-}
-
 template <typename T, int VEC>
 __global__ void activation_kernel(const T* x, int x_stride, int x_col, T* out, int out_stride, int out_col, int per_row, long long total,
                                   int kind, float cap) {
@@ -530,7 +523,7 @@ __global__ void activation_kernel(const T* x, int x_stride, int x_col, T* out, i
         const int c = (int)(idx - t * per_row) * VEC;
         Pack p = *reinterpret_cast<const Pack*>(x + t * x_stride + x_col + c);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(activate(to_f32<T>(p.v[e]), kind, cap));
+        for (int e = 0; e < VEC; ++e) p.v[e] = from_f32<T>(unary_activation(to_f32<T>(p.v[e]), kind, cap));
         *reinterpret_cast<Pack*>(out + t * out_stride + out_col + c) = p;
     }
 }

@@ -61,7 +61,7 @@ __device__ __forceinline__ uint4 ld_stream(const void* p, uint64_t policy) {
 
 static inline int blocks_wanted() { return 2 * kvb_sm_count(); }     // two blocks an SM
 
-enum { EPI_PLAIN = 0, EPI_ACT = 1, EPI_RESID = 2, EPI_ROPE = 3 };
+enum { EPI_PLAIN = 0, EPI_ACT = 1, EPI_RESID = 2, EPI_ROPE = 3, EPI_UNARY = 4 };
 
 // What the fused forms need beyond x, W, bias and y.
 struct Fused {
@@ -81,6 +81,7 @@ struct Fused {
     int* err;
     int table_len, table_stride, Hq, Hkv, D, page_size, page_shift, writes;
     float act_limit;          // EPI_ACT: 0 - silu(g) * u; > 0 - the clamped gated activation with this limit (common.cuh)
+    int unary, ldy;           // EPI_UNARY: y[m * ldy + n] = unary_activation(., unary)
 };
 
 __device__ __forceinline__ void unpack8(const uint4& v, float (&f)[8]) {
@@ -364,6 +365,12 @@ __global__ void __maxnreg__((RT == 1 && NT <= 2) ? 96 : 255) gemm_skinny_kernel(
                     if (m + e < M) y[(size_t)(m + e) * I + i] = from_f32<TOut>(gated_pair(gate, up, fz.act_limit));
                 }
             }
+        } else if (EPI == EPI_UNARY) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int nn = n + 8 * (e >> 1), mm = m + (e & 1);
+                if (nn < N && mm < M) y[(size_t)mm * fz.ldy + nn] = from_f32<TOut>(unary_activation(vals[e], fz.unary, 0.f));
+            }
         } else if (EPI == EPI_RESID) {
             float hv[4];
 #pragma unroll
@@ -556,6 +563,18 @@ KVB_API int kvb_gemm_skinny_gated(int out_dtype, const void* x, const void* w, v
                                   cudaStream_t stream) {
     if (!(limit > 0.f)) return KVB_ERR_SHAPE;
     return gemm_skinny(out_dtype, 1, x, w, nullptr, y, M, N, K, limit, stream);
+}
+
+// The product with an activation of one number in its epilogue (unary_activation, kinds 1 and 3), into N columns of rows of `ldy`
+// numbers: M <= 16, bfloat16.
+KVB_API int kvb_gemm_skinny_unary(int kind, const void* x, const void* w, void* y, int ldy, int M, int N, int K, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return KVB_OK;
+    if (M > 16 || K <= 0 || K % 32 != 0 || ldy < N || (kind != 1 && kind != 3)) return KVB_ERR_SHAPE;
+    if (((uintptr_t)x | (uintptr_t)w) & 15) return KVB_ERR_ALIGN;
+    skinny::Fused fz = {};
+    fz.unary = kind;
+    fz.ldy = ldy;
+    return skinny::dispatch<skinny::EPI_UNARY, false, bf16>((const bf16*)x, (const bf16*)w, nullptr, (bf16*)y, M, N, K, K, fz, stream);
 }
 
 // The fused forms (M <= 16, bfloat16 throughout).  `x` holds rows of the residual stream rounded to bfloat16 where

@@ -196,6 +196,7 @@ _SIGNATURES = {
     "gemm_skinny": {
         "kvb_gemm_skinny": [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_gemm_skinny_gated": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+        "kvb_gemm_skinny_unary": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_gemm_skinny_norm_act": [_c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_gemm_skinny_residual": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
         "kvb_gemm_skinny_qkv": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p,
@@ -706,6 +707,26 @@ class CudaKernels(KernelSet):
         self._count("gemm_simt")
         _check(self._gemm_simt.kvb_gemm_simt(_dtype_code(x.dtype), _dtype_code(out.dtype), _ptr(x), _ptr(w),
                                              _ptr(bias), _ptr(out), M, N, K, self._stream()), "linear")
+
+    def linear_act(self, x: torch.Tensor, w: torch.Tensor, kind: str, out: torch.Tensor, out_col: int, workspace) -> None:
+        """out[:, out_col : out_col + N] = act(x . w^T), act "relu2" or "gelu" (see `activation_`): in the product's epilogue for
+        steps of few rows, else the product and then the activation."""
+        M, (N, K) = x.shape[0], w.shape
+        if kind not in ("relu2", "gelu") or x.shape[1] != K or out.shape[0] != M or out_col + N > out.shape[1]:
+            raise KernelError(f"linear_act: x{tuple(x.shape)} w{tuple(w.shape)} '{kind}' out{tuple(out.shape)} at {out_col} do not fit")
+        if out.dtype == torch.bfloat16 and M <= 16 and self._skinny(x.dtype, M, K, N):
+            self._count("gemm_skinny")
+            _ptr(out)                                        # a contiguous tensor on the device, as for every operand
+            _check(self._gemm_skinny.kvb_gemm_skinny_unary(self.ACTIVATIONS[kind], _ptr(x), _ptr(w), _c_void_p(out.data_ptr() + 2 * out_col),
+                                                           out.shape[1], M, N, K, self._stream()), "linear_act (skinny)")
+            return
+        if out_col == 0 and out.shape[1] == N:
+            self.linear(x, w, out)
+            self.activation_(out, kind)
+            return
+        act = workspace.buffer("linear.act", (M, N), out.dtype)
+        self.linear(x, w, act)
+        self.activation_into(act, kind, out, out_col)
 
     def qkv_rope_append(self, qkv: torch.Tensor, bias: Optional[torch.Tensor], cos: Optional[torch.Tensor],
                         sin: Optional[torch.Tensor], batch: StepBatch, kv: PagedKVView, q_out: torch.Tensor,

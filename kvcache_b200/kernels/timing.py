@@ -46,7 +46,7 @@ def _attention_bytes(batch, kv, num_heads: int, reach=None) -> int:
 
 
 class KernelTiming:
-    OPERATORS = ("embed", "add_rmsnorm", "silu_mul", "gate_up_act", "linear", "qkv_rope_append", "rope_append_attention",
+    OPERATORS = ("embed", "add_rmsnorm", "silu_mul", "gate_up_act", "linear", "linear_act", "qkv_rope_append", "rope_append_attention",
                  "paged_attention", "sample", "norm_add_rmsnorm", "latent_norm_rope_append", "head_linear", "latent_attention",
                  "route_top", "route_sigmoid", "routed_experts", "bigram_embed", "head_gate", "head_norm_gate", "gated_linear_scan",
                  "matrix_memory_scan", "token_shift", "activation_", "activation_into", "delta_rule_scan", "lightning_scan",
@@ -65,6 +65,9 @@ class KernelTiming:
         if name == "linear":
             x, w, out = args[0], args[1], args[2]
             return f"linear {w.shape[0]}x{w.shape[1]}", _numel_bytes(w) + _numel_bytes(x) + _numel_bytes(out)
+        if name == "linear_act":
+            x, w = args[0], args[1]
+            return f"linear_act {w.shape[0]}x{w.shape[1]}", _numel_bytes(w) + _numel_bytes(x) + x.shape[0] * w.shape[0] * x.element_size()
         if name == "gate_up_act":
             x, w, out = args[0], args[1], args[2]
             return f"gate_up_act {w.shape[0]}x{w.shape[1]}", _numel_bytes(w) + _numel_bytes(x) + _numel_bytes(out)
@@ -179,7 +182,7 @@ class KernelTiming:
     @classmethod
     def _flops(cls, name: str, args, kwargs) -> int:
         """Multiply-adds times two that the call's matrix products need (0 for classes that are only moved bytes)."""
-        if name == "linear":
+        if name in ("linear", "linear_act"):
             return 2 * args[0].shape[0] * args[1].shape[0] * args[1].shape[1]
         if name == "gate_up_act":
             return 2 * args[0].shape[0] * args[1].shape[0] * args[1].shape[1]

@@ -125,16 +125,13 @@ class PlainMLP(FeedForward):
 
     def forward_hidden(self, x: torch.Tensor, ctx: LayerContext, out: torch.Tensor, out_col: int = 0) -> None:
         """act(Wup x) into columns out_col .. out_col + hidden_width of `out`."""
-        act = ctx.workspace.buffer("ffn.act", (x.shape[0], self.intermediate), self.dtype)
-        ctx.kernels.linear(x, self.w_up, act)
-        ctx.kernels.activation_into(act, self.activation, out, out_col)
+        ctx.kernels.linear_act(x, self.w_up, self.activation, out, out_col, ctx.workspace)
 
     def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
         T = x.shape[0]
         k, ws = ctx.kernels, ctx.workspace
         act = ws.buffer("ffn.act", (T, self.intermediate), self.dtype)
-        k.linear(x, self.w_up, act)
-        k.activation_(act, self.activation)
+        k.linear_act(x, self.w_up, self.activation, act, 0, ws)
         delta = ws.buffer("ffn.delta", (T, self.hidden), self.dtype)
         k.linear(act, self.w_down, delta)
         return delta

@@ -83,6 +83,24 @@ def test_activation_into_columns_of_wider_rows(kernels, dtype, kind, cols, wide,
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("kind", ["gelu", "relu2"])
+@pytest.mark.parametrize("M", [1, 3, 8, 13, 16, 17, 40, 300])
+@pytest.mark.parametrize("N,K,wide,at", [(192, 128, 400, 104), (50, 96, 50, 0), (45, 40, 77, 11), (4864, 896, 6656, 1792)])
+def test_product_with_an_activation(kernels, dtype, kind, M, N, K, wide, at):
+    """Into columns of wider rows: in the product's epilogue for few rows (bfloat16, K in steps of 32), else in two launches."""
+    from kvcache_b200.engine.workspace import Workspace
+    x, w = _rand(M, K, dtype=dtype, seed=1), _rand(N, K, dtype=dtype, seed=2, scale=0.2)
+    ref, got = torch.full((M, wide), 5.0).to(dtype), torch.full((M, wide), 5.0).to(dtype).to(DEV)
+    TorchKernels(wide=True).linear_act(x, w, kind, ref, at)
+    before = kernels.launches
+    kernels.linear_act(x.to(DEV), w.to(DEV), kind, got, at, Workspace(DEV))
+    if dtype == torch.bfloat16 and K % 32 == 0:
+        assert kernels.launches - before == (1 if M <= 16 else 2)
+    assert_close(got, ref, TOL[dtype])
+    assert bool((got[:, :at] == 5.0).all()) and bool((got[:, at + N:] == 5.0).all())
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("per_channel", [True, False, None])
 @pytest.mark.parametrize("H,Dv,xs,g_col,wide,at", [(3, 16, 16, 8, 80, 16), (4, 5, 9, 3, 40, 7), (14, 64, 64, 1152, 6656, 0), (2, 48, 64, 0, 96, 0)])
 def test_head_gate_per_head_and_per_channel(kernels, dtype, per_channel, H, Dv, xs, g_col, wide, at):

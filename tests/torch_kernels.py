@@ -482,6 +482,10 @@ class TorchKernels:
     def activation_into(self, x, kind, out, out_col=0, cap=0.0):
         out[:, out_col:out_col + x.shape[1]] = self._activated(x.to(self.f), kind, cap).to(out.dtype)
 
+    def linear_act(self, x, w, kind, out, out_col, workspace=None):
+        y = x.to(self.f) @ w.to(self.f).t()
+        out[:, out_col:out_col + w.shape[0]] = self._activated(y, kind, 0.0).to(out.dtype)
+
     # ---- operators of the short convolutions, the gated delta rule and the state-space mixer ------------------------------
     def _short_conv(self, x, conv_w, conv_b, tail, batch):
         """silu(bias + sum_n w[n] x_{t - (taps - 1) + n}) per segment; tail[slot] holds the inputs before the segment's first."""
