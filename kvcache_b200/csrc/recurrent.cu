@@ -668,6 +668,9 @@ static int scan_any(int mode, const float* proj, int P, int q_col, int k_col, in
     // lane took 312 us where 128 took 489 and 32 took 475; at 64 key channels one lane a column 129 us, four 160);
     // fewer lanes where the exponential-gate form's block (all of a head's columns) would pass 16 warps.
     int ks = D <= 64 ? 1 : D <= 128 ? 2 : 4;
+    // The gated delta rule, which holds more beside the state: two lanes from 33 key channels on (2,048 rows, 14 heads of 64: 235 us
+    // against 321).
+    if (mode == SCAN_GATED_DELTA && D > 32 && D <= 64) ks = 2;
     if (scan_mixes_keys(mode) && delta_rule_lanes > 0) ks = delta_rule_lanes;
     if (mode == SCAN_EXP_GATES)
         while (ks > 1 && (Dv + 32 / ks - 1) / (32 / ks) > 16) ks >>= 1;

@@ -1413,10 +1413,11 @@ class CudaKernels(KernelSet):
             float(unit_eps), _ptr(rows), _ptr(gates), gates.shape[1], _ptr(batch.row_segment), _ptr(batch.seg_q_start), _ptr(batch.seg_q_len),
             _ptr(batch.seg_slot), T, batch.num_segments, H, G, D, Dv, self._stream()), "gated_delta_inputs")
 
-    # Portions of at least this many rows go through the scan that spreads a column over many lanes (csrc/scan_wide.cu): the state
-    # space always, the gated delta rule where a head has more key channels than DELTA_WIDE_ABOVE - with fewer, chunks that run side
-    # by side are ahead (2,048 rows, 14 heads of 64: 313 us in chunks, 478 us; 16 heads of 128: 810 us in chunks, 462 us).
-    SCAN_WIDE_MIN_ROWS = 64
+    # Portions of at least SCAN_WIDE_MIN_ROWS rows go through the scan that spreads a column over many lanes (csrc/scan_wide.cu):
+    # the state space always (28 heads of 128 x 64: 40 us at 64 rows in one piece, 15 us), the gated delta rule where a head has more
+    # key channels than DELTA_WIDE_ABOVE (2,048 rows, 16 heads of 128: 818 us in chunks, 454 us); with fewer, portions long enough
+    # for chunks that run side by side take those (14 heads of 64: 235 us at 2,048 rows, 527 us).
+    SCAN_WIDE_MIN_ROWS = 48
     DELTA_WIDE_ABOVE = 64
 
     def gated_delta_scan(self, rows: torch.Tensor, gates: torch.Tensor, q_scale: float, batch: StepBatch, memory: torch.Tensor,
@@ -1428,12 +1429,13 @@ class CudaKernels(KernelSet):
             raise KernelError(f"the gated delta scan wants states [slots, {H}, {D}, {Dv}], got {tuple(memory.shape)}")
         segments = (_ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_slot), _ptr(memory), _ptr(out))
         self._count("gated_delta_scan")
-        if D > self.DELTA_WIDE_ABOVE and batch.max_q_len >= self.SCAN_WIDE_MIN_ROWS:
+        chunked = self.SCAN_CHUNK and batch.max_q_len >= self.SCAN_CHUNK_MIN_ROWS
+        if batch.max_q_len >= self.SCAN_WIDE_MIN_ROWS and (D > self.DELTA_WIDE_ABOVE or not chunked):
             _check(self._scan_wide.kvb_gated_delta_scan_wide(_ptr(rows), _ptr(gates), gates.shape[1], float(q_scale), *segments,
                                                              batch.num_segments, H, G, D, Dv, self._stream()), "gated_delta_scan (wide)")
             return
         max_chunks, scratch, chunk = 0, None, self.SCAN_CHUNK
-        if chunk and batch.max_q_len >= self.SCAN_CHUNK_MIN_ROWS:
+        if chunked:
             if batch.max_q_len >= self.DELTA_LONG_ROWS:
                 chunk = max(chunk, self.DELTA_LONG_CHUNK)
             max_chunks = -(-batch.num_tokens // chunk) + batch.num_segments          # as in `delta_rule_scan`

@@ -224,11 +224,12 @@ def test_scans(kernels, kind, H, G, D, Dv):
 @pytest.mark.parametrize("kind", ["delta", "space"])
 @pytest.mark.parametrize("H,G,D,Dv", [(4, 2, 64, 64), (1, 1, 33, 40), (2, 1, 128, 64), (3, 3, 8, 12), (2, 2, 200, 48), (2, 2, 128, 128), (2, 1, 100, 45),
                                        (3, 1, 70, 5), (1, 1, 256, 33)])
-def test_scans_of_long_portions(kernels, kind, H, G, D, Dv):
+@pytest.mark.parametrize("shorter", [False, True])
+def test_scans_of_long_portions(kernels, kind, H, G, D, Dv, shorter):
     """Portions for the scan that spreads a column over many lanes and for the one in chunks: many tiles of tokens, from an empty
     state and from a filled one, lengths that are no multiple of a tile or a group, beside single tokens and short portions;
     against the plain recurrence, and every segment alone, which must give the same bits (in the forms without chunks)."""
-    segments, slots = [(0, 300), (50, 1), (100, 257), (3, 1), (0, 64), (5, 2)], [2, 0, 3, 5, 1, 4]
+    segments, slots = [(0, 120 if shorter else 300), (50, 1), (100, 97 if shorter else 257), (3, 1), (0, 64), (5, 2)], [2, 0, 3, 5, 1, 4]
     batch = _segments_batch(segments, slots)
     T = batch.num_tokens
     rows, gates = (_delta_rows if kind == "delta" else _space_rows)(T, H, G, D, Dv)
@@ -242,7 +243,7 @@ def test_scans_of_long_portions(kernels, kind, H, G, D, Dv):
     assert_close(got, want, 1e-4, "read-out")
     assert_close(got_mem, ref_mem, 1e-4, "states")
     assert torch.equal(got_mem[6].cpu(), memory[6])
-    if kind == "space" or D > kernels.DELTA_WIDE_ABOVE:
+    if kind == "space" or D > kernels.DELTA_WIDE_ABOVE or shorter:
         at, alone_mem = 0, memory.clone().to(DEV)
         for (start, n), slot in zip(segments, slots):
             if n >= kernels.SCAN_WIDE_MIN_ROWS:
@@ -259,14 +260,14 @@ def test_forms_of_the_delta_scan_agree(kernels, D):
     segments = [(0, 300), (4, 70)]
     rows, gates = (t.to(DEV) for t in _delta_rows(370, H, G, D, Dv))
     batch = batch_to(_segments_batch(segments, [1, 0]), DEV)
-    saved, results = (kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK), []
+    saved, results = (kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK, kernels.SCAN_WIDE_MIN_ROWS), []
     try:
-        for above, chunk in ((0, 64), (256, 64), (256, 0)):
-            kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK = above, chunk
+        for above, chunk, rows_wide in ((0, 64, 48), (256, 64, 48), (256, 0, 1 << 30)):
+            kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK, kernels.SCAN_WIDE_MIN_ROWS = above, chunk, rows_wide
             memory = _rand(2, H, D, Dv, seed=3).to(DEV)
             results.append((_run_scan(kernels, "delta", rows, gates, batch, memory, (H, G, D, Dv)), memory))
     finally:
-        kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK = saved
+        kernels.DELTA_WIDE_ABOVE, kernels.SCAN_CHUNK, kernels.SCAN_WIDE_MIN_ROWS = saved
     for out, memory in results[1:]:
         assert_close(out, results[0][0], 1e-5)
         assert_close(memory, results[0][1], 1e-5)
